@@ -5,5 +5,6 @@ from .buzetar import BuzetarConfig
 from .kisepel import KisepelConfig
 from .zamizen import ZamizenConfig
 from .nomutar import NomutarConfig
+from .fipadra import FipadraConfig
 
-__all__ = ["ConfigError", "ModelConfig", "Rule", "apply_rules", "read_config_json", "Qwen3Config", "YarnScaling", "BuzetarConfig", "KisepelConfig", "ZamizenConfig", "NomutarConfig"]
+__all__ = ["ConfigError", "ModelConfig", "Rule", "apply_rules", "read_config_json", "Qwen3Config", "YarnScaling", "BuzetarConfig", "KisepelConfig", "ZamizenConfig", "NomutarConfig", "FipadraConfig"]

@@ -7,9 +7,12 @@
 //                        row order, whatever else the launch holds); then one block cuts the lists into tiles of
 //                        32 or 128 pairs (as the products' form wants): (expert, first place in the list), compactly,
 //                        with their number.
-//   llmx_moe_gate_up     act[pair, f] = silu(h[row] . Wg_e[f]) * (h[row] . Wu_e[f])         (gate and up rows stacked per expert)
-//   llmx_moe_down        y[pair, c]   = act[pair] . Wd_e[c]                                 (32-bit)
+//   llmx_moe_product     gated: act[pair, f] = glu(h[row] . Wg_e[f], h[row] . Wu_e[f])       (gate and up rows stacked per expert;
+//                        glu(g, u) = silu(g) u, or the clamped unit min(g, L) sigmoid(alpha min(g, L)) (clamp(u, -L, L) + 1));
+//                        else y[pair, c] = act[pair] . Wd_e[c]                               (32-bit)
 //   llmx_moe_combine     x[row]      += weight * sum_k y[row * top + k]                      (k in order: one order of sums)
+// A pair may name an expert beyond those that have weights (an identity expert): it is in no list, the products leave its
+// rows alone, and `llmx_moe_combine_weighted` takes the row's input in its place.
 // The products run one block a (tile of an expert's pairs, tile of output columns): rows are gathered through the
 // list, the expert's weights are read once a tile.  Two forms: on the CUDA cores with explicit fmaf and k in
 // increasing order (32-bit weights and rows: the true 32-bit path; also bfloat16 shapes the tensor-core form does not
@@ -21,6 +24,18 @@
 
 namespace {
 constexpr int TILE_ROWS = 32;     // pairs a tile holds
+
+// The gated unit of an expert: silu(g) * u without a clamp, else the clamped one.
+struct Glu {
+    int clamped;
+    float limit, alpha;
+};
+__device__ __forceinline__ float glu_f(const Glu& a, float g, float u) {
+    if (!a.clamped) return g / (1.0f + expf(-g)) * u;
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g / (1.0f + expf(-a.alpha * g)) * (u + 1.0f);
+}
 
 __global__ void __launch_bounds__(256)
 route_kernel(const int* __restrict__ token_ids, const int* __restrict__ table, int top, int rows, int experts, int vocab,
@@ -83,7 +98,7 @@ template <typename T, bool GATED, typename OutT>
 __global__ void __launch_bounds__(256)
 moe_cores_kernel(const T* __restrict__ a, int a_div, const T* __restrict__ w, const int* __restrict__ lists,
                  const int* __restrict__ counts, const int* __restrict__ tiles, int pairs, OutT* __restrict__ out, int N,
-                 int K) {
+                 int K, Glu glu) {
     pdl_trigger();
     pdl_wait();
     if ((int)blockIdx.x >= tiles[0] || tiles[1] != TILE_ROWS) return;
@@ -138,7 +153,7 @@ moe_cores_kernel(const T* __restrict__ a, int a_div, const T* __restrict__ w, co
             const int c = col0 + tc + 16 * j;
             if (c >= N) continue;
             float v = acc[i][j];
-            if (GATED) v = v / (1.0f + expf(-v)) * acc2[i][j];
+            if (GATED) v = glu_f(glu, v, acc2[i][j]);
             out[(size_t)p * N + c] = from_float<OutT>(v);
         }
     }
@@ -148,7 +163,7 @@ moe_cores_kernel(const T* __restrict__ a, int a_div, const T* __restrict__ w, co
 // A block of eight warps: a tile of 128 pairs (the routing cut the lists into tiles of 128 for this form) x 128 weight
 // rows, K in steps of 32 through four stages of cp.async copies (16-byte pieces; rows that do not exist are filled with
 // zeros by the copy itself).  The 128 weight rows are two halves of 64: gated, the gate rows and the up rows of the
-// same 64 output columns, so that a thread holds both of an output and writes silu(gate) * up; else 128 output columns.
+// same 64 output columns, so that a thread holds both of an output and writes the gated unit; else 128 output columns.
 // The weights are the A operand of mma.sync m16n8k16 and the gathered rows the B operand, both read by ldmatrix from
 // rows padded by 8 values (no two of a read's eight rows in one bank).  Warp (wm, wn), wm < 4, wn < 2: weight rows
 // 16 wm .. of both halves x pairs 64 wn .. 64 wn + 63.
@@ -171,7 +186,7 @@ template <bool GATED, typename OutT>
 __global__ void __launch_bounds__(256)
 moe_tc_kernel(const __nv_bfloat16* __restrict__ a, int a_div, const __nv_bfloat16* __restrict__ w,
               const int* __restrict__ lists, const int* __restrict__ counts, const int* __restrict__ tiles, int pairs,
-              OutT* __restrict__ out, int N, int K) {
+              OutT* __restrict__ out, int N, int K, Glu glu) {
     pdl_trigger();
     pdl_wait();
     if ((int)blockIdx.x >= tiles[0] || tiles[1] != TC_ROWS) return;
@@ -278,10 +293,7 @@ moe_tc_kernel(const __nv_bfloat16* __restrict__ a, int a_div, const __nv_bfloat1
             if (p < 0) continue;
             if (GATED) {
                 const int c = col0 + rr;
-                if (c < N) {
-                    const float g = acc[0][t][i];
-                    out[(size_t)p * N + c] = from_float<OutT>(g / (1.0f + expf(-g)) * acc[1][t][i]);
-                }
+                if (c < N) out[(size_t)p * N + c] = from_float<OutT>(glu_f(glu, acc[0][t][i], acc[1][t][i]));
             } else {
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
@@ -314,7 +326,7 @@ template <bool GATED, typename OutT>
 __global__ void __launch_bounds__(256)
 moe_few_kernel(const __nv_bfloat16* __restrict__ a, int a_div, const __nv_bfloat16* __restrict__ w,
                const int* __restrict__ token_ids, const int* __restrict__ table, int top, int vocab, int experts,
-               OutT* __restrict__ out, int N, int K) {
+               OutT* __restrict__ out, int N, int K, Glu glu) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char few_smem[];
@@ -343,7 +355,7 @@ moe_few_kernel(const __nv_bfloat16* __restrict__ a, int a_div, const __nv_bfloat
         }
         s0 = warp_sum(s0);
         if (GATED) s1 = warp_sum(s1);
-        if (lane == 0) out[(size_t)p * N + c] = from_float<OutT>(GATED ? s0 / (1.0f + expf(-s0)) * s1 : s0);
+        if (lane == 0) out[(size_t)p * N + c] = from_float<OutT>(GATED ? glu_f(glu, s0, s1) : s0);
     }
 }
 
@@ -360,25 +372,34 @@ __global__ void combine_kernel(const float* __restrict__ y, float* __restrict__ 
     x[i] = fmaf(weight, s, x[i]);
 }
 
-// x[row] += factor * sum_k pair_weight[row * top + k] * y[row * top + k], k in increasing order.
-__global__ void combine_weighted_kernel(const float* __restrict__ y, float* __restrict__ x, const float* __restrict__ pair_weight,
-                                        int top, int width, float factor, long long n) {
-    pdl_trigger();
-    pdl_wait();
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= n) return;
-    const long long row = i / width;
-    const int c = (int)(i % width);
-    float s = 0.0f;
-    for (int k = 0; k < top; ++k) s = fmaf(pair_weight[row * top + k], y[((size_t)row * top + k) * width + c], s);
-    x[i] = fmaf(factor, s, x[i]);
-}
+// A router: logits z = h W^T + b in 32-bit (h may be bfloat16; the weights are 32-bit) and from them a choice of `top`
+// outputs (the lower index first among equals) and their weights, in one of two ways:
+//   over the chosen   the largest logits; weights: the softmax over the chosen logits alone
+//   over all          s = softmax over all outputs; the largest s + correction among the outputs that may be chosen; weights:
+//                     s / (sum of the chosen s + 1e-20) * scale.  With `group_keep` < `group_count` the outputs form equal
+//                     groups of neighbours and only members of the groups with the largest best s + correction may be chosen
+// `extra` more rows of W after the outputs' give one number a row each through a sigmoid (a gate on a part that runs beside
+// the experts).  A block takes R rows of the step (1 when the rows are few, so that they spread over the SMs; 8 when they
+// are many, so that a weight row is read once for 8 rows); a row's logits do not depend on what else the step holds.
+struct RouterChoice {
+    int over_all, group_count, group_keep;
+    const float* correction;
+    float scale;
+};
 
-// A router: logits z = h W^T + b in 32-bit (h may be bfloat16; the weights are 32-bit), the `top` largest (the lower index
-// first among equals), and as weights the softmax over the chosen logits alone.  `extra` more rows of W after the experts'
-// give one number a row each through a sigmoid (a gate on a part that runs beside the experts).  A block takes R rows of
-// the step (1 when the rows are few, so that they spread over the SMs; 8 when they are many, so that a weight row is read
-// once for 8 rows); a row's logits do not depend on what else the step holds.
+// The best of v[0 .. n) over a warp: (value, index), the lower index among equals; index -1 when none exceeds minus infinity.
+__device__ __forceinline__ void warp_best(const float* v, int n, int lane, float& bv, int& bi) {
+    bv = -INFINITY;
+    bi = -1;
+    for (int e = lane; e < n; e += 32)
+        if (v[e] > bv) bv = v[e], bi = e;                    // no number is never larger
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > bv || (ov == bv && oi >= 0 && (bi < 0 || oi < bi))) bv = ov, bi = oi;
+    }
+}
 __device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
     const float4 t = *reinterpret_cast<const float4*>(p);
     v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w;
@@ -393,7 +414,7 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&v)[4]) {
 template <typename T, int R, int VEC>
 __global__ void __launch_bounds__(256)
 router_kernel(const T* __restrict__ h, const float* __restrict__ w, const float* __restrict__ bias, int rows, int K, int experts,
-              int top, int extra, int* __restrict__ choice, float* __restrict__ weight, float* __restrict__ gate) {
+              int top, int extra, RouterChoice rule, int* __restrict__ choice, float* __restrict__ weight, float* __restrict__ gate) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float router_z[];                    // [R][experts + extra], then the warps' parts [8][experts + extra][R]
@@ -457,59 +478,160 @@ router_kernel(const T* __restrict__ h, const float* __restrict__ w, const float*
         const int r = i / extra, x = i - r * extra;
         if (row0 + r < rows) gate[(size_t)(row0 + r) * extra + x] = 1.0f / (1.0f + expf(-router_z[r * outs + experts + x]));
     }
-    if (threadIdx.x >= R || row0 + (int)threadIdx.x >= rows) return;
-    // One thread a row picks: the largest logit left, `top` times (a chosen one is struck out in shared memory; the chosen
-    // logits wait in the warps' parts, which nobody reads any more), then the softmax over the chosen.
-    float* z = router_z + threadIdx.x * outs;
-    float* picked = part + (size_t)threadIdx.x * top;
-    int* mine = choice + (size_t)(row0 + threadIdx.x) * top;
-    float* wt = weight + (size_t)(row0 + threadIdx.x) * top;
-    for (int k = 0; k < top; ++k) {
-        int best = -1;
-        float bz = -INFINITY;
-        for (int e = 0; e < experts; ++e) {
-            const float ze = z[e];
-            if (ze > bz) best = e, bz = ze;                  // the lower index first among equals; no number is never larger
+    // A warp a row picks (R is at most the block's warps).  The warps' parts, which nobody reads any more, hold the row's
+    // choice scores, the picked values and the groups' best scores.
+    if (warp >= R || row0 + warp >= rows) return;
+    float* z = router_z + warp * outs;                       // logits; over all: scores
+    float* cs = part + (size_t)warp * 8 * outs;              // choice scores; a chosen one is struck out
+    float* picked = cs + outs;
+    float* best_of = picked + outs;
+    int* mine = choice + (size_t)(row0 + warp) * top;
+    float* wt = weight + (size_t)(row0 + warp) * top;
+    if (rule.over_all) {
+        float zmax = -INFINITY;
+        for (int e = lane; e < experts; e += 32) zmax = fmaxf(zmax, z[e]);
+        zmax = warp_max(zmax);
+        float sum = 0.0f;
+        for (int e = lane; e < experts; e += 32) {
+            z[e] = expf(z[e] - zmax);
+            sum += z[e];
         }
+        sum = warp_sum(sum);
+        for (int e = lane; e < experts; e += 32) {
+            z[e] /= sum;
+            cs[e] = z[e] + (rule.correction ? rule.correction[e] : 0.0f);
+        }
+        __syncwarp();
+        if (rule.group_keep < rule.group_count) {
+            const int size = experts / rule.group_count;
+            for (int g = lane; g < rule.group_count; g += 32) {
+                float b = -INFINITY;
+                for (int i = 0; i < size; ++i) b = fmaxf(b, cs[g * size + i]);
+                best_of[g] = b;
+            }
+            __syncwarp();
+            for (int n = 0; n < rule.group_keep; ++n) {      // a kept group is marked by plus infinity once all lanes have looked
+                float b = -INFINITY;
+                int bi = -1;
+                for (int g = lane; g < rule.group_count; g += 32)
+                    if (best_of[g] > b && best_of[g] < INFINITY) b = best_of[g], bi = g;
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, b, o);
+                    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+                    if (ob > b || (ob == b && oi >= 0 && (bi < 0 || oi < bi))) b = ob, bi = oi;
+                }
+                __syncwarp();
+                if (lane == 0 && bi >= 0) best_of[bi] = INFINITY;
+                __syncwarp();
+            }
+            for (int e = lane; e < experts; e += 32)
+                if (best_of[e / size] != INFINITY) cs[e] = -INFINITY;
+            __syncwarp();
+        }
+    } else {
+        for (int e = lane; e < experts; e += 32) cs[e] = z[e];
+        __syncwarp();
+    }
+    for (int k = 0; k < top; ++k) {
+        float bv;
+        int best;
+        warp_best(cs, experts, lane, bv, best);
         if (best < 0) {                                      // nothing left that is a number
             for (int e = 0; e < experts && best < 0; ++e)
-                if (z[e] != z[e]) best = e;
+                if (cs[e] != cs[e]) best = e;
             best = best < 0 ? 0 : best;
         }
-        z[best] = -INFINITY;
-        mine[k] = best;
-        picked[k] = bz;
+        __syncwarp();
+        if (lane == 0) {
+            mine[k] = best;
+            picked[k] = rule.over_all ? z[best] : bv;
+            cs[best] = -INFINITY;
+        }
+        __syncwarp();
     }
+    if (lane != 0) return;
+    float sum = rule.over_all ? 1e-20f : 0.0f;
     const float zmax = picked[0];
-    float sum = 0.0f;
     for (int k = 0; k < top; ++k) {
-        const float e = zmax == -INFINITY ? 1.0f : expf(picked[k] - zmax);
-        picked[k] = e;
-        sum += e;
+        if (!rule.over_all) picked[k] = zmax == -INFINITY ? 1.0f : expf(picked[k] - zmax);
+        sum += picked[k];
     }
-    for (int k = 0; k < top; ++k) wt[k] = picked[k] / sum;
+    for (int k = 0; k < top; ++k) wt[k] = picked[k] / sum * (rule.over_all ? rule.scale : 1.0f);
+}
+
+// x[row] += factor * sum_k pair_weight[row * top + k] * e_k + shared_gate[row] * shared[row], k in increasing order: e_k is
+// the expert's output y[row * top + k], or, when `choice` names an expert beyond the `experts` that have weights, the row's
+// input h[row].  `choice` null: every pair has an expert's output.  `shared` null: no such part.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+combine_weighted_kernel(const float* __restrict__ y, float* __restrict__ x, const float* __restrict__ pair_weight,
+                        const int* __restrict__ choice, int experts, const T* __restrict__ h, const float* __restrict__ shared,
+                        const float* __restrict__ shared_gate, int top, int width, float factor, long long pieces) {
+    pdl_trigger();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= pieces) return;
+    const int per_row = width / VEC;
+    const long long row = i / per_row;
+    const int c = (int)(i - row * per_row) * VEC;
+    auto read = [](auto* p, float (&v)[VEC]) {
+        if constexpr (VEC == 4) load4(p, v);
+        else v[0] = to_float(*p);
+    };
+    float s[VEC], v[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) s[j] = 0.0f;
+    for (int k = 0; k < top; ++k) {
+        const long long p = row * top + k;
+        const float w = pair_weight[p];
+        if (choice && choice[p] >= experts) read(h + (size_t)row * width + c, v);
+        else read(y + (size_t)p * width + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) s[j] = fmaf(w, v[j], s[j]);
+    }
+    float* dst = x + (size_t)row * width + c;
+    float t[VEC];
+    read(dst, t);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) t[j] = fmaf(factor, s[j], t[j]);
+    if (shared) {
+        const float g = shared_gate[row];
+        read(shared + (size_t)row * width + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) t[j] = fmaf(g, v[j], t[j]);
+    }
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst) = make_float4(t[0], t[1], t[2], t[3]);
+    else dst[0] = t[0];
 }
 
 inline int max_tiles(int pairs, int experts, int tile_rows) { return (pairs + tile_rows - 1) / tile_rows + experts; }
 }  // namespace
 
-// h [rows, K] of `dtype`; w float32 [experts + extra, K]; bias float32 [experts] or null; choice int32 [rows, top]; weight float32
-// [rows, top]; gate float32 [rows, extra] (extra 0: not used).
-LLMX_EXPORT int llmx_moe_router(const void* h, int dtype, const float* w, const float* bias, int rows, int K, int experts, int top,
-                                int extra, int* choice, float* weight, float* gate, cudaStream_t stream) {
+// h [rows, K] of `dtype`; w float32 [outputs + extra, K]; bias float32 [outputs] or null; choice int32 [rows, top]; weight float32
+// [rows, top]; gate float32 [rows, extra] (extra 0: not used).  `over_all` 0: weights are the softmax over the chosen logits;
+// 1: scores over all outputs, with `correction` [outputs] (or null) counting for the choice alone, `group_keep` of
+// `group_count` groups, and `scale` on the weights.
+LLMX_EXPORT int llmx_moe_router(const void* h, int dtype, const float* w, const float* bias, int rows, int K, int outputs, int top,
+                                int extra, int over_all, const float* correction, int group_count, int group_keep, float scale,
+                                int* choice, float* weight, float* gate, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (K <= 0 || experts <= 0 || top <= 0 || top > experts || extra < 0 || extra > 128 || (extra > 0 && gate == nullptr) ||
-        experts + extra > 1024)
+    if (K <= 0 || outputs <= 0 || top <= 0 || top > outputs || extra < 0 || extra > 128 || (extra > 0 && gate == nullptr) ||
+        outputs + extra > 1024)
         return LLMX_ERR_BAD_ARGUMENT;
+    if (over_all && (group_count <= 0 || outputs % group_count || group_keep <= 0 || group_keep > group_count ||
+                     top > group_keep * (outputs / group_count)))
+        return LLMX_ERR_BAD_ARGUMENT;
+    const RouterChoice rule = {over_all, group_count, group_keep, correction, scale};
     // Eight rows a block when the rows are many (a weight row is then read once for eight rows), one when they are few.
     const bool vec = (K & 3) == 0 && !((uintptr_t)h & 15) && !((uintptr_t)w & 15);
     int R = rows > 64 ? 8 : 1;
-    size_t smem = (size_t)9 * R * (experts + extra) * sizeof(float);
-    if (smem > 40 * 1024) R = 1, smem = (size_t)9 * (experts + extra) * sizeof(float);
+    size_t smem = (size_t)9 * R * (outputs + extra) * sizeof(float);
+    if (smem > 40 * 1024) R = 1, smem = (size_t)9 * (outputs + extra) * sizeof(float);
     if (smem > 40 * 1024) return LLMX_ERR_UNSUPPORTED;
     const dim3 grid((rows + R - 1) / R);
 #define LLMX_ROUTER(T, RR, V) \
-    launch_kernel(router_kernel<T, RR, V>, grid, dim3(256), smem, stream, (const T*)h, w, bias, rows, K, experts, top, extra, choice, weight, gate)
+    launch_kernel(router_kernel<T, RR, V>, grid, dim3(256), smem, stream, (const T*)h, w, bias, rows, K, outputs, top, extra, rule, choice, weight, gate)
 #define LLMX_ROUTER_T(T)                      \
     do {                                      \
         if (R == 8 && vec) LLMX_ROUTER(T, 8, 4); \
@@ -525,13 +647,25 @@ LLMX_EXPORT int llmx_moe_router(const void* h, int dtype, const float* w, const 
     return launch_status();
 }
 
-// x [rows, width] += factor * sum over k of pair_weight[rows * top] * y [rows * top, width], k in increasing order.
-LLMX_EXPORT int llmx_moe_combine_weighted(const float* y, float* x, const float* pair_weight, int rows, int top, int width,
-                                          float factor, cudaStream_t stream) {
+// x [rows, width] += factor * sum over k of pair_weight[rows * top] * (y [rows * top, width], or h [rows, width] of `h_dtype` where
+// choice[rows * top] >= experts), k in increasing order, + shared_gate[rows] * shared [rows, width].  choice and h, shared and
+// shared_gate: null when the design has no such experts, no such part.
+LLMX_EXPORT int llmx_moe_combine_weighted(const float* y, float* x, const float* pair_weight, const int* choice, int experts,
+                                          const void* h, int h_dtype, const float* shared, const float* shared_gate, int rows,
+                                          int top, int width, float factor, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (pair_weight == nullptr) return LLMX_ERR_BAD_ARGUMENT;
-    const long long n = (long long)rows * width;
-    launch_kernel(combine_weighted_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, y, x, pair_weight, top, width, factor, n);
+    if (pair_weight == nullptr || top <= 0 || width <= 0 || (choice && h == nullptr) || (shared && shared_gate == nullptr))
+        return LLMX_ERR_BAD_ARGUMENT;
+    const bool vec = width % 4 == 0 && !(((uintptr_t)y | (uintptr_t)x | (uintptr_t)h | (uintptr_t)shared) & 15);
+    const long long pieces = (long long)rows * (vec ? width / 4 : width);
+    const dim3 grid((unsigned)((pieces + 255) / 256));
+#define LLMX_COMBINE(T, V) \
+    launch_kernel(combine_weighted_kernel<T, V>, grid, dim3(256), 0, stream, y, x, pair_weight, choice, experts, (const T*)h, shared, shared_gate, top, width, factor, pieces)
+    if (h_dtype == LLMX_BF16 && vec) LLMX_COMBINE(__nv_bfloat16, 4);
+    else if (h_dtype == LLMX_BF16) LLMX_COMBINE(__nv_bfloat16, 1);
+    else if (vec) LLMX_COMBINE(float, 4);
+    else LLMX_COMBINE(float, 1);
+#undef LLMX_COMBINE
     return launch_status();
 }
 
@@ -555,14 +689,15 @@ LLMX_EXPORT int llmx_moe_route(const int* token_ids, const int* table, int top, 
 }
 
 // a [rows of `a_div` pairs each, K] and w [experts, (gated ? 2 : 1) * N, K] of `dtype`; out [pairs, N] of `out_dtype`
-// (gated: silu(gate) * up; else the plain product, float32).  `tensor_cores`: the form to run; the routing must have cut
+// (gated: silu(gate) * up, or the clamped unit of `limit` and `alpha` if `clamped`; else the plain product, float32).  `tensor_cores`: the form to run; the routing must have cut
 // the lists into tiles of `llmx_moe_tile_rows(tensor_cores)` pairs.
 LLMX_EXPORT int llmx_moe_product(const void* a, int a_div, const void* w, int dtype, const int* lists, const int* counts,
                                  const int* tiles, int pairs, int experts, void* out, int out_dtype, int N, int K,
-                                 int gated, int tensor_cores, cudaStream_t stream) {
+                                 int gated, int clamped, float limit, float alpha, int tensor_cores, cudaStream_t stream) {
     if (pairs <= 0) return 0;
     if (N <= 0 || K <= 0 || a_div <= 0) return LLMX_ERR_BAD_ARGUMENT;
     if (!gated && out_dtype != LLMX_F32) return LLMX_ERR_UNSUPPORTED;
+    const Glu glu = {clamped, limit, alpha};
     if (tensor_cores) {
         if (!llmx_moe_tensor_cores_fit(dtype, K) || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return LLMX_ERR_UNSUPPORTED;
         const int out_cols = gated ? TC_HALF : 2 * TC_HALF;
@@ -574,7 +709,7 @@ LLMX_EXPORT int llmx_moe_product(const void* a, int a_div, const void* w, int dt
     do {                                                                                                                \
         cudaFuncSetAttribute(moe_tc_kernel<G, O>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM);          \
         launch_kernel(moe_tc_kernel<G, O>, dim3(grid), dim3(256), TC_SMEM, stream, ab, a_div, wb, lists, counts, tiles, \
-                      pairs, (O*)out, N, K);                                                                            \
+                      pairs, (O*)out, N, K, glu);                                                                          \
     } while (0)
         if (gated && out_dtype == LLMX_BF16) LLMX_MOE_TC(true, __nv_bfloat16);
         else if (gated) LLMX_MOE_TC(true, float);
@@ -585,7 +720,7 @@ LLMX_EXPORT int llmx_moe_product(const void* a, int a_div, const void* w, int dt
     dim3 grid(max_tiles(pairs, experts, TILE_ROWS), (N + CC_COLS - 1) / CC_COLS);
     if (grid.y > 65535) return LLMX_ERR_UNSUPPORTED;
 #define LLMX_MOE(T, G, O) \
-    launch_kernel(moe_cores_kernel<T, G, O>, dim3(grid), dim3(256), 0, stream, (const T*)a, a_div, (const T*)w, lists, counts, tiles, pairs, (O*)out, N, K)
+    launch_kernel(moe_cores_kernel<T, G, O>, dim3(grid), dim3(256), 0, stream, (const T*)a, a_div, (const T*)w, lists, counts, tiles, pairs, (O*)out, N, K, glu)
     if (dtype == LLMX_BF16 && gated && out_dtype == LLMX_BF16) LLMX_MOE(__nv_bfloat16, true, __nv_bfloat16);
     else if (dtype == LLMX_BF16 && gated && out_dtype == LLMX_F32) LLMX_MOE(__nv_bfloat16, true, float);
     else if (dtype == LLMX_BF16 && !gated) LLMX_MOE(__nv_bfloat16, false, float);
@@ -600,10 +735,11 @@ LLMX_EXPORT int llmx_moe_product(const void* a, int a_div, const void* w, int dt
 // multiple of 8; the pair's expert is read from the table.
 LLMX_EXPORT int llmx_moe_product_few(const void* a, int a_div, const void* w, const int* token_ids, const int* table,
                                      int top, int vocab, int pairs, int experts, void* out, int out_dtype, int N, int K,
-                                     int gated, cudaStream_t stream) {
+                                     int gated, int clamped, float limit, float alpha, cudaStream_t stream) {
     if (pairs <= 0) return 0;
     if (N <= 0 || K <= 0 || K % 8 || a_div <= 0 || top <= 0 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return LLMX_ERR_UNSUPPORTED;
     if (!gated && out_dtype != LLMX_F32) return LLMX_ERR_UNSUPPORTED;
+    const Glu glu = {clamped, limit, alpha};
     const size_t smem = (size_t)K * 2;
     if (smem > 200 * 1024) return LLMX_ERR_UNSUPPORTED;
     dim3 grid(pairs, (N + GV_COLS - 1) / GV_COLS);
@@ -612,7 +748,7 @@ LLMX_EXPORT int llmx_moe_product_few(const void* a, int a_div, const void* w, co
     do {                                                                                                                \
         if (smem > 48 * 1024) cudaFuncSetAttribute(moe_few_kernel<G, O>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         launch_kernel(moe_few_kernel<G, O>, dim3(grid), dim3(256), smem, stream, (const __nv_bfloat16*)a, a_div,       \
-                      (const __nv_bfloat16*)w, token_ids, table, top, vocab, experts, (O*)out, N, K);                   \
+                      (const __nv_bfloat16*)w, token_ids, table, top, vocab, experts, (O*)out, N, K, glu);              \
     } while (0)
     if (gated && out_dtype == LLMX_BF16) LLMX_FEW(true, __nv_bfloat16);
     else if (gated) LLMX_FEW(true, float);

@@ -156,6 +156,98 @@ LLMX_EXPORT int llmx_rmsnorm(const float* x, const float* w, void* y, int out_dt
 }
 
 // ---------------------------------------------------------------------------
+// Two RMS norms of one row with one epsilon: y1 = x * (r * w1), y2 = x * (r * w2), r = 1 / sqrt(mean(x^2) + eps) made
+// once.  (A block whose mixer and feed-forward read the same stream through norms of their own.)  One block a row; blocks
+// beyond the rows clear `zero`, as in RMSNorm.  The row stays in registers when it fits (REGS), else it is read again.
+// ---------------------------------------------------------------------------
+template <typename OutT, bool REGS>
+__global__ void rmsnorm_pair_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
+                                    OutT* __restrict__ y1, OutT* __restrict__ y2, int rows, int width, float eps,
+                                    float* __restrict__ zero, long long zero_count) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int r = blockIdx.x;
+    if (r >= rows) {
+        float4* z = reinterpret_cast<float4*>(zero);
+        const long long n4 = zero_count >> 2;
+        const long long blocks = gridDim.x - rows;
+        for (long long i = (long long)(r - rows) * blockDim.x + threadIdx.x; i < n4; i += blocks * blockDim.x)
+            z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        return;
+    }
+    const size_t base = (size_t)r * width;
+    if constexpr (REGS) {
+        const float4* src = reinterpret_cast<const float4*>(x + base);
+        const float4* wa = reinterpret_cast<const float4*>(w1);
+        const float4* wb = reinterpret_cast<const float4*>(w2);
+        const int n4 = width >> 2;
+        float4 v[NORM_VEC_MAX];
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            v[k] = i < n4 ? src[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        float s = 0.0f;
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            s = fmaf(v[k].x, v[k].x, s);
+            s = fmaf(v[k].y, v[k].y, s);
+            s = fmaf(v[k].z, v[k].z, s);
+            s = fmaf(v[k].w, v[k].w, s);
+        }
+        s = block_sum(s, scratch);
+        const float rr = 1.0f / sqrtf(s / (float)width + eps);
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < n4) {
+                const float4 a = wa[i], b = wb[i];
+                store4(y1 + base + 4 * i, v[k].x * (rr * a.x), v[k].y * (rr * a.y), v[k].z * (rr * a.z), v[k].w * (rr * a.w));
+                store4(y2 + base + 4 * i, v[k].x * (rr * b.x), v[k].y * (rr * b.y), v[k].z * (rr * b.z), v[k].w * (rr * b.w));
+            }
+        }
+    } else {
+        float s = 0.0f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) s = fmaf(x[base + i], x[base + i], s);
+        s = block_sum(s, scratch);
+        const float rr = 1.0f / sqrtf(s / (float)width + eps);
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            const float v = x[base + i];
+            y1[base + i] = from_float<OutT>(v * (rr * w1[i]));
+            y2[base + i] = from_float<OutT>(v * (rr * w2[i]));
+        }
+    }
+}
+
+// The block width that a norm over rows of `width` values uses: it depends on the width alone, so that a row's sum has one
+// order whatever the batch.
+static inline int norm_threads(int width) {
+    int threads = ((width / 4 + 3) / 4 + 31) / 32 * 32;
+    return threads < 32 ? 32 : threads > 256 ? 256 : threads;
+}
+
+LLMX_EXPORT int llmx_rmsnorm_pair(const float* x, const float* w1, const float* w2, void* y1, void* y2, int out_dtype, int rows,
+                                  int width, float eps, float* zero, long long zero_count, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (width <= 0 || (zero && (zero_count % 4 || ((uintptr_t)zero & 15)))) return LLMX_ERR_BAD_ARGUMENT;
+    const bool regs = width % 4 == 0 && width <= 4 * NORM_VEC_MAX * 256 &&
+                      !(((uintptr_t)x | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)y1 | (uintptr_t)y2) & 15);
+    const int threads = regs ? norm_threads(width) : width >= 1024 ? 256 : 128;
+    long long zero_blocks = zero ? (zero_count / 4 + 4 * threads - 1) / (4 * threads) : 0;
+    zero_blocks = zero_blocks > 1024 ? 1024 : zero_blocks;
+    const dim3 grid((unsigned)(rows + zero_blocks));
+#define LLMX_PAIR(O, R) \
+    launch_kernel(rmsnorm_pair_kernel<O, R>, grid, dim3(threads), 0, stream, x, w1, w2, (O*)y1, (O*)y2, rows, width, eps, zero, zero_count)
+    if (out_dtype == LLMX_BF16 && regs) LLMX_PAIR(__nv_bfloat16, true);
+    else if (out_dtype == LLMX_BF16) LLMX_PAIR(__nv_bfloat16, false);
+    else if (regs) LLMX_PAIR(float, true);
+    else LLMX_PAIR(float, false);
+#undef LLMX_PAIR
+    return launch_status();
+}
+
+// ---------------------------------------------------------------------------
 // Per-head norm, rotation and cache write, one warp per (row, head).
 //
 // For a query head: RMSNorm over the head's D values with q_weight (skipped when null),
@@ -424,6 +516,44 @@ LLMX_EXPORT int llmx_embed_scaled(const void* table, int table_dtype, const int*
     return launch_status();
 }
 
+// ---------------------------------------------------------------------------
+// Embedding with a norm: z = table[ids[r], :] * scale; x[r, :] = z / sqrt(mean(z^2) + eps) * w, 32-bit.  One block a row;
+// the second pass finds the row in the caches.
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x, int width,
+                                  int table_rows, float scale, const float* __restrict__ w, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int id = ids[blockIdx.x];
+    float* dst = x + (size_t)blockIdx.x * width;
+    if (id < 0 || id >= table_rows) {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = 0.0f;
+        return;
+    }
+    const T* src = table + (size_t)id * width;
+    float s = 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = to_float(src[i]) * scale;
+        s = fmaf(v, v, s);
+    }
+    s = block_sum(s, scratch);
+    const float rr = 1.0f / sqrtf(s / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = to_float(src[i]) * scale * (rr * w[i]);
+}
+
+LLMX_EXPORT int llmx_embed_norm(const void* table, int table_dtype, const int* ids, float* x, int rows, int width, int table_rows,
+                                float scale, const float* w, float eps, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (w == nullptr) return LLMX_ERR_BAD_ARGUMENT;
+    if (table_dtype == LLMX_BF16)
+        launch_kernel(embed_norm_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, (const __nv_bfloat16*)table, ids, x, width, table_rows, scale, w, eps);
+    else
+        launch_kernel(embed_norm_kernel<float>, dim3(rows), dim3(256), 0, stream, (const float*)table, ids, x, width, table_rows, scale, w, eps);
+    return launch_status();
+}
+
 // x[i] *= s over a flat float buffer (a model whose logits carry a factor).
 __global__ void scale_kernel(float* __restrict__ x, long long n, float s) {
     pdl_trigger();
@@ -616,6 +746,86 @@ LLMX_EXPORT int llmx_clamped_glu(const float* gu, void* act, int out_dtype, int 
 }
 
 // ---------------------------------------------------------------------------
+// The square of relu: act = max(x, 0)^2, 32-bit arithmetic.
+// ---------------------------------------------------------------------------
+__device__ __forceinline__ float relu2_f(float v) {
+    const float m = fmaxf(v, 0.0f);
+    return m * m;
+}
+
+template <typename OutT, int VEC>
+__global__ void relu_squared_kernel(const float* __restrict__ x, OutT* __restrict__ act, long long pieces) {
+    pdl_trigger();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= pieces) return;
+    if constexpr (VEC == 4) {
+        const float4 v = reinterpret_cast<const float4*>(x)[i];
+        store4(act + 4 * i, relu2_f(v.x), relu2_f(v.y), relu2_f(v.z), relu2_f(v.w));
+    } else {
+        act[i] = from_float<OutT>(relu2_f(x[i]));
+    }
+}
+
+LLMX_EXPORT int llmx_relu_squared(const float* x, void* act, int out_dtype, long long n, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    const bool vec = n % 4 == 0 && !(((uintptr_t)x | (uintptr_t)act) & 15);
+    const long long pieces = vec ? n / 4 : n;
+    const dim3 grid((unsigned)((pieces + 255) / 256));
+    if (out_dtype == LLMX_BF16 && vec) launch_kernel(relu_squared_kernel<__nv_bfloat16, 4>, grid, dim3(256), 0, stream, x, (__nv_bfloat16*)act, pieces);
+    else if (out_dtype == LLMX_BF16) launch_kernel(relu_squared_kernel<__nv_bfloat16, 1>, grid, dim3(256), 0, stream, x, (__nv_bfloat16*)act, pieces);
+    else if (vec) launch_kernel(relu_squared_kernel<float, 4>, grid, dim3(256), 0, stream, x, (float*)act, pieces);
+    else launch_kernel(relu_squared_kernel<float, 1>, grid, dim3(256), 0, stream, x, (float*)act, pieces);
+    return launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// In-place rotation of q and k heads inside a projection's rows: columns 0 .. (q_heads + k_heads) * D - 1 are heads of D
+// values, q heads first.  Pair (i, i + rot_dims / 2), i < rot_dims / 2, of every head is turned by p * freq_i (p: the row's
+// position; the cosines and sines are made once a row, in shared memory); then every value of a q head is multiplied by
+// q_factor and of a k head by k_factor.  Angles and arithmetic are 32-bit.  A block makes one row.
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+rotate_heads_kernel(float* __restrict__ x, int stride, int q_heads, int k_heads, int D, int half, const float* __restrict__ freq,
+                    const int* __restrict__ positions, float q_factor, float k_factor) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ float turn[];                  // cosines [half], sines [half]
+    float* row = x + (size_t)blockIdx.x * stride;
+    const float p = (float)positions[blockIdx.x];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(p * freq[i], &turn[half + i], &turn[i]);
+    __syncthreads();
+    const int heads = q_heads + k_heads;
+    for (int e = threadIdx.x; e < heads * half; e += blockDim.x) {
+        const int h = e / half, i = e - h * half;
+        float* v = row + (size_t)h * D + i;
+        const float f = h < q_heads ? q_factor : k_factor;
+        const float c = turn[i], s = turn[half + i], a = v[0], b = v[half];
+        v[0] = (a * c - b * s) * f;
+        v[half] = (b * c + a * s) * f;
+    }
+    const int rest = D - 2 * half;                   // the values that pass unturned still take the factor
+    if (rest > 0 && (q_factor != 1.0f || k_factor != 1.0f))
+        for (int e = threadIdx.x; e < heads * rest; e += blockDim.x) {
+            const int h = e / rest;
+            row[(size_t)h * D + 2 * half + (e - h * rest)] *= h < q_heads ? q_factor : k_factor;
+        }
+}
+
+LLMX_EXPORT int llmx_rotate_heads(float* x, int rows, int stride, int q_heads, int k_heads, int D, int rot_dims, const float* freq,
+                                  const int* positions, float q_factor, float k_factor, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (q_heads < 0 || k_heads < 0 || D <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > D || (rot_dims > 0 && freq == nullptr) ||
+        (long long)(q_heads + k_heads) * D > stride)
+        return LLMX_ERR_BAD_ARGUMENT;
+    const size_t smem = (size_t)rot_dims * sizeof(float);
+    if (smem > 48 * 1024) return LLMX_ERR_UNSUPPORTED;
+    launch_kernel(rotate_heads_kernel, dim3(rows), dim3(256), smem, stream, x, stride, q_heads, k_heads, D, rot_dims / 2, freq, positions,
+                  q_factor, k_factor);
+    return launch_status();
+}
+
+// ---------------------------------------------------------------------------
 // In-place activation of a column range of a float matrix: x[r, c0 .. c0 + n) = silu(x).  (A mixer whose
 // projections pass an activation before a recurrence reads them.)
 // ---------------------------------------------------------------------------
@@ -641,9 +851,56 @@ LLMX_EXPORT int llmx_silu_columns(float* x, int rows, int stride, int c0, int n,
 // RMS norm over groups of a row, times a gate: for group j of `group` values,
 //   y = o / sqrt(mean_group(o^2) + eps) * w[(j * group + i) % w_len] * act(gate),  act = sigmoid (0) or silu (1).
 // One group is the whole row (a norm over all heads together, weight as long as the row) or one head (weight as
-// long as a head and shared by the heads).  `gate` has its own row stride (it lies inside a wider product's output).
-// One block per (row, group); the block width follows the group width alone.
+// long as a head and shared by the heads); w null: no weight.  `gate` has its own row stride (it lies inside a wider
+// product's output).  Two forms, chosen by the group width and the alignment alone: heads of up to 512 values, a warp a
+// (row, group) with the values in registers and 16-byte accesses; else one block per (row, group), whose width follows
+// the group width.
 // ---------------------------------------------------------------------------
+template <typename OutT, int PIECES>
+__global__ void __launch_bounds__(256)
+gated_rmsnorm_warp_kernel(const float* __restrict__ o, const float* __restrict__ gate, int gate_stride, const float* __restrict__ w,
+                          int w_len, OutT* __restrict__ y, int rows, int groups, int group, float eps, int gate_kind) {
+    pdl_trigger();
+    pdl_wait();
+    const long long unit = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (unit >= (long long)rows * groups) return;
+    const int lane = threadIdx.x & 31, n4 = group >> 2;
+    const long long r = unit / groups;
+    const int j = (int)(unit - r * groups);
+    const float4* src = reinterpret_cast<const float4*>(o + (size_t)unit * group);
+    const float4* gsrc = reinterpret_cast<const float4*>(gate + (size_t)r * gate_stride + (size_t)j * group);
+    const float4* wsrc = w ? reinterpret_cast<const float4*>(w + (size_t)j * group % w_len) : nullptr;
+    const float4 none = make_float4(0.f, 0.f, 0.f, 0.f), ones = make_float4(1.f, 1.f, 1.f, 1.f);
+    float4 v[PIECES], g[PIECES];
+#pragma unroll
+    for (int k = 0; k < PIECES; ++k) {
+        const int i = lane + 32 * k;
+        v[k] = i < n4 ? src[i] : none;
+        g[k] = i < n4 ? gsrc[i] : none;
+    }
+    float s = 0.0f;
+#pragma unroll
+    for (int k = 0; k < PIECES; ++k) {
+        s = fmaf(v[k].x, v[k].x, s);
+        s = fmaf(v[k].y, v[k].y, s);
+        s = fmaf(v[k].z, v[k].z, s);
+        s = fmaf(v[k].w, v[k].w, s);
+    }
+    const float rr = 1.0f / sqrtf(warp_sum(s) / (float)group + eps);
+    auto act = [&](float z) {
+        const float sg = 1.0f / (1.0f + expf(-z));
+        return gate_kind == 0 ? sg : z * sg;
+    };
+#pragma unroll
+    for (int k = 0; k < PIECES; ++k) {
+        const int i = lane + 32 * k;
+        if (i >= n4) continue;
+        const float4 ww = wsrc ? wsrc[i] : ones;
+        store4(y + (size_t)unit * group + 4 * i, v[k].x * rr * ww.x * act(g[k].x), v[k].y * rr * ww.y * act(g[k].y),
+               v[k].z * rr * ww.z * act(g[k].z), v[k].w * rr * ww.w * act(g[k].w));
+    }
+}
+
 template <typename OutT>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int gate_stride,
                                      const float* __restrict__ w, int w_len, OutT* __restrict__ y, int groups, int group,
@@ -667,7 +924,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
     const float rr = 1.0f / sqrtf(block_sum(s, scratch) / (float)group + eps);
     for (int i = threadIdx.x; i < group; i += blockDim.x) {
         const float a = act(gsrc[i]);
-        const float wi = w[(j * group + i) % w_len];
+        const float wi = w ? w[(j * group + i) % w_len] : 1.0f;
         y[base + i] = from_float<OutT>(gate_first ? (src[i] * a) * rr * wi : src[i] * rr * wi * a);
     }
 }
@@ -677,7 +934,24 @@ LLMX_EXPORT int llmx_gated_rmsnorm(const float* o, const float* gate, int gate_s
                                    int out_dtype, int rows, int groups, int group, float eps, int gate_kind, int gate_first,
                                    cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (groups <= 0 || group <= 0 || w_len <= 0 || groups > 65535 || (gate_kind != 0 && gate_kind != 1)) return LLMX_ERR_BAD_ARGUMENT;
+    if (groups <= 0 || group <= 0 || (w && w_len <= 0) || groups > 65535 || (gate_kind != 0 && gate_kind != 1)) return LLMX_ERR_BAD_ARGUMENT;
+    if (groups > 1 && group <= 512 && group % 4 == 0 && gate_stride % 4 == 0 && !gate_first && (!w || w_len % group == 0) &&
+        !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)y) & 15)) {
+        const dim3 grid((unsigned)(((long long)rows * groups + 7) / 8));
+#define LLMX_GATED(O, P) \
+    launch_kernel(gated_rmsnorm_warp_kernel<O, P>, grid, dim3(256), 0, stream, o, gate, gate_stride, w, w_len, (O*)y, rows, groups, group, eps, gate_kind)
+        if (out_dtype == LLMX_BF16) {
+            if (group <= 128) LLMX_GATED(__nv_bfloat16, 1);
+            else if (group <= 256) LLMX_GATED(__nv_bfloat16, 2);
+            else LLMX_GATED(__nv_bfloat16, 4);
+        } else {
+            if (group <= 128) LLMX_GATED(float, 1);
+            else if (group <= 256) LLMX_GATED(float, 2);
+            else LLMX_GATED(float, 4);
+        }
+#undef LLMX_GATED
+        return launch_status();
+    }
     int threads = (group + 3) / 4;
     threads = (threads + 31) / 32 * 32;
     threads = threads < 32 ? 32 : threads > 256 ? 256 : threads;

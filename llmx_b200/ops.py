@@ -95,6 +95,10 @@ _SIGNATURES = {
                                             _i, _i, _i, _i, _i, _p],
     ("rowwise", "llmx_swiglu"): [_p, _p, _i, _i, _i, _p],
     ("rowwise", "llmx_embed_scaled"): [_p, _i, _p, _p, _i, _i, _i, _f, _p],
+    ("rowwise", "llmx_embed_norm"): [_p, _i, _p, _p, _i, _i, _i, _f, _p, _f, _p],
+    ("rowwise", "llmx_rmsnorm_pair"): [_p, _p, _p, _p, _p, _i, _i, _i, _f, _p, ctypes.c_longlong, _p],
+    ("rowwise", "llmx_relu_squared"): [_p, _p, _i, ctypes.c_longlong, _p],
+    ("rowwise", "llmx_rotate_heads"): [_p, _i, _i, _i, _i, _i, _i, _p, _p, _f, _f, _p],
     ("rowwise", "llmx_scale"): [_p, ctypes.c_longlong, _f, _p],
     ("rowwise", "llmx_layernorm"): [_p, _p, _p, _i, _p, _i, _i, _f, _p, ctypes.c_longlong, _p],
     ("rowwise", "llmx_layernorm_affine"): [_p, _p, _p, _p, _p, _i, _p, _f, _p, _i, _i, _f, _p, ctypes.c_longlong, _p],
@@ -121,11 +125,11 @@ _SIGNATURES = {
     ("attention_split", "llmx_attention_tiled"): [_p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f,
                                                   _f, _p, _i, _p, _i, _p],
     ("moe", "llmx_moe_route"): [_p, _p, _i, _i, _i, _i, _p, _p, _p, _i, _p],
-    ("moe", "llmx_moe_product_few"): [_p, _i, _p, _p, _p, _i, _i, _i, _i, _p, _i, _i, _i, _i, _p],
-    ("moe", "llmx_moe_product"): [_p, _i, _p, _i, _p, _p, _p, _i, _i, _p, _i, _i, _i, _i, _i, _p],
+    ("moe", "llmx_moe_product_few"): [_p, _i, _p, _p, _p, _i, _i, _i, _i, _p, _i, _i, _i, _i, _i, _f, _f, _p],
+    ("moe", "llmx_moe_product"): [_p, _i, _p, _i, _p, _p, _p, _i, _i, _p, _i, _i, _i, _i, _i, _f, _f, _i, _p],
     ("moe", "llmx_moe_combine"): [_p, _p, _i, _i, _i, _f, _p],
-    ("moe", "llmx_moe_router"): [_p, _i, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p, _p],
-    ("moe", "llmx_moe_combine_weighted"): [_p, _p, _p, _i, _i, _i, _f, _p],
+    ("moe", "llmx_moe_router"): [_p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _p, _p, _p, _p],
+    ("moe", "llmx_moe_combine_weighted"): [_p, _p, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _f, _p],
     ("rowwise", "llmx_group_norm_conv"): [_p, _p, _i, _i, _f, _p, _i, _p, _p, _i, _p, _i, _p, ctypes.c_longlong, ctypes.c_longlong,
                                           _p, _p, _p, _p, _p, _p, _i, _p, ctypes.c_longlong, _p],
     ("rowwise", "llmx_embed_pairs"): [_p, _p, _i, _p, _p, _i, _i, _i, _f, _i, ctypes.c_longlong, ctypes.c_longlong, _p, _p, _p, _p, _p,
@@ -251,6 +255,21 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
     return out
 
 
+def rmsnorm_pair(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor, eps: float, out1: torch.Tensor, out2: torch.Tensor,
+                 zero: Optional[torch.Tensor] = None) -> None:
+    """out1 = x / sqrt(mean x^2 + eps) * w1 and out2 the same with w2, row by row in one launch; x float32, outputs of one
+    type.  `zero` as in `rmsnorm`."""
+    _cuda(x, w1, w2, out1, out2, zero)
+    rows, width = x.shape
+    _need(zero is None or (zero.dtype == torch.float32 and zero.numel() % 4 == 0), "rmsnorm_pair: the buffer to clear must be float32, a multiple of 4 long")
+    _need(x.dtype == torch.float32 and all(w.dtype == torch.float32 and w.numel() == width for w in (w1, w2)),
+          "rmsnorm_pair: float32 rows and two float32 weights of their width")
+    _need(tuple(out1.shape) == (rows, width) and tuple(out2.shape) == (rows, width) and out1.dtype == out2.dtype,
+          "rmsnorm_pair: two outputs of the input's shape and one type")
+    _check(_fn("rowwise", "llmx_rmsnorm_pair")(_ptr(x), _ptr(w1), _ptr(w2), _ptr(out1), _ptr(out2), _code(out1), rows, width, float(eps),
+                                               _ptr(zero), 0 if zero is None else zero.numel(), _stream()), "rmsnorm_pair")
+
+
 def head_norm_rope_kv(qkv: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                       q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                       cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor,
@@ -342,6 +361,40 @@ def embed_scaled(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scal
     return out
 
 
+def embed_norm(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """z = table[ids[r], :] * scale; out[r] = z / sqrt(mean z^2 + eps) * weight, in float32."""
+    _cuda(table, ids, out, weight)
+    rows, width = out.shape
+    _need(ids.dtype == torch.int32 and ids.numel() == rows, "embed: ids must be int32, one per output row")
+    _need(out.dtype == torch.float32 and table.dim() == 2 and table.shape[1] == width and weight.dtype == torch.float32
+          and weight.numel() == width, "embed: shapes do not fit")
+    _check(_fn("rowwise", "llmx_embed_norm")(_ptr(table), _code(table), _ptr(ids), _ptr(out), rows, width, table.shape[0], float(scale),
+                                             _ptr(weight), float(eps), _stream()), "embed_norm")
+    return out
+
+
+def relu_squared(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = max(x, 0)^2; x float32, out float32 or bfloat16 of the same shape."""
+    _cuda(x, out)
+    _need(x.dtype == torch.float32 and out.shape == x.shape, "relu_squared: float32 input, an output of its shape")
+    _check(_fn("rowwise", "llmx_relu_squared")(_ptr(x), _ptr(out), _code(out), x.numel(), _stream()), "relu_squared")
+    return out
+
+
+def rotate_heads_(x: torch.Tensor, q_heads: int, k_heads: int, head_dim: int, rot_dims: int, freq: Optional[torch.Tensor],
+                  positions: torch.Tensor, q_factor: float = 1.0, k_factor: float = 1.0) -> torch.Tensor:
+    """The first (q_heads + k_heads) * head_dim columns of x float32 [rows, width], in place: pair (i, i + rot_dims / 2) of every
+    head turned by position * freq_i (freq float32 [rot_dims / 2]), then q heads times q_factor and k heads times k_factor."""
+    _cuda(x, freq, positions)
+    _need(x.dtype == torch.float32 and x.dim() == 2 and (q_heads + k_heads) * head_dim <= x.shape[1], "rotate_heads: heads inside float32 rows")
+    _need(positions.dtype == torch.int32 and positions.numel() >= x.shape[0], "rotate_heads: an int32 position per row")
+    _need(rot_dims % 2 == 0 and 0 <= rot_dims <= head_dim and (rot_dims == 0 or (freq is not None and freq.dtype == torch.float32
+          and freq.numel() == rot_dims // 2)), "rotate_heads: an even rotated width and a float32 frequency per pair")
+    _check(_fn("rowwise", "llmx_rotate_heads")(_ptr(x), x.shape[0], x.shape[1], q_heads, k_heads, head_dim, rot_dims, _ptr(freq),
+                                               _ptr(positions), float(q_factor), float(k_factor), _stream()), "rotate_heads")
+    return x
+
+
 def scale_(x: torch.Tensor, factor: float) -> torch.Tensor:
     """x *= factor in place; x float32."""
     _cuda(x)
@@ -428,21 +481,22 @@ def silu_columns_(x: torch.Tensor, first: int, count: int) -> torch.Tensor:
     return x
 
 
-def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, group: int, gate_kind: str,
+def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float, group: int, gate_kind: str,
                   out: torch.Tensor, gate_first: bool = False) -> torch.Tensor:
     """out = o / sqrt(mean over each group of `group` values of o^2 + eps) * weight * act(gate); act sigmoid or silu.
     `gate_first`: the gate comes before the norm: z = o * act(gate), out = z / sqrt(mean z^2 + eps) * weight.
     o float32 [rows, width] contiguous; gate float32 [rows, width], a view whose rows may be strided; weight float32 of
-    the row's width, or of one group's width and shared by the groups."""
-    _need(o.is_cuda and gate.is_cuda and weight.is_cuda and out.is_cuda, "kernel arguments must be CUDA tensors (there is no CPU path)")
+    the row's width, or of one group's width and shared by the groups, or None for a norm without a weight."""
+    _cuda(weight)
+    _need(o.is_cuda and gate.is_cuda and out.is_cuda, "kernel arguments must be CUDA tensors (there is no CPU path)")
     rows, width = o.shape
-    _need(o.is_contiguous() and out.is_contiguous() and weight.is_contiguous(), "gated_rmsnorm: contiguous input, weight and output")
-    _need(o.dtype == torch.float32 and gate.dtype == torch.float32 and weight.dtype == torch.float32, "gated_rmsnorm: float32 inputs")
+    _need(o.is_contiguous() and out.is_contiguous(), "gated_rmsnorm: contiguous input and output")
+    _need(o.dtype == torch.float32 and gate.dtype == torch.float32 and (weight is None or weight.dtype == torch.float32), "gated_rmsnorm: float32 inputs")
     _need(tuple(out.shape) == (rows, width) and tuple(gate.shape) == (rows, width) and gate.stride(1) == 1, "gated_rmsnorm: shapes do not fit")
-    _need(group > 0 and width % group == 0 and weight.numel() in (group, width), "gated_rmsnorm: the group must divide the row; weight of a group or of the row")
+    _need(group > 0 and width % group == 0 and (weight is None or weight.numel() in (group, width)), "gated_rmsnorm: the group must divide the row; weight of a group or of the row")
     _need(gate_kind in ("sigmoid", "silu"), "gated_rmsnorm: gate must be sigmoid or silu")
     _check(_fn("rowwise", "llmx_gated_rmsnorm")(_ptr(o), _ptr(gate), gate.stride(0) if rows > 1 else width, _ptr(weight),
-                                                weight.numel(), _ptr(out), _code(out), rows, width // group, group,
+                                                0 if weight is None else weight.numel(), _ptr(out), _code(out), rows, width // group, group,
                                                 float(eps), 0 if gate_kind == "sigmoid" else 1, 1 if gate_first else 0, _stream()),
            "gated_rmsnorm")
     return out
@@ -820,10 +874,16 @@ def moe_tensor_cores_fit(dtype: torch.dtype, *inner_widths: int) -> bool:
     return dtype in _CODE and all(bool(f(_CODE[dtype], int(k))) for k in inner_widths)
 
 
+def _clamp(clamp):
+    """(clamped, limit, alpha) of an expert's gated unit: None for silu(gate) * up."""
+    return (0, 0.0, 0.0) if clamp is None else (1, float(clamp[0]), float(clamp[1]))
+
+
 def moe_product_few(a: torch.Tensor, a_div: int, w: torch.Tensor, token_ids: torch.Tensor, table: torch.Tensor, pairs: int,
-                    out: torch.Tensor, gated: bool) -> torch.Tensor:
+                    out: torch.Tensor, gated: bool, clamp=None) -> torch.Tensor:
     """`moe_product` for steps of a few pairs (bfloat16, inner width a multiple of 8): a block a pair and 16 output
     columns, the pair's expert read from the table, no lists."""
+    clamped, limit, alpha = _clamp(clamp)
     _cuda(a, w, token_ids, table, out)
     experts, wn, K = w.shape
     N = wn // 2 if gated else wn
@@ -836,7 +896,8 @@ def moe_product_few(a: torch.Tensor, a_div: int, w: torch.Tensor, token_ids: tor
           "moe_product_few: int32 ids and table")
     _need(tuple(out.shape) == (pairs, N), "moe_product_few: output shape does not fit")
     _check(_fn("moe", "llmx_moe_product_few")(_ptr(a), int(a_div), _ptr(w), _ptr(token_ids), _ptr(table), top, vocab, pairs, experts,
-                                              _ptr(out), _code(out), N, K, 1 if gated else 0, _stream()), "moe_product_few")
+                                              _ptr(out), _code(out), N, K, 1 if gated else 0, clamped, limit, alpha, _stream()),
+           "moe_product_few")
     return out
 
 
@@ -862,27 +923,36 @@ def moe_route(token_ids: torch.Tensor, table: torch.Tensor, experts: int, lists:
 
 
 def moe_product(a: torch.Tensor, a_div: int, w: torch.Tensor, lists: torch.Tensor, counts: torch.Tensor, tiles: torch.Tensor,
-                pairs: int, out: torch.Tensor, gated: bool, tensor_cores: bool = False) -> torch.Tensor:
+                pairs: int, out: torch.Tensor, gated: bool, tensor_cores: bool = False, clamp=None) -> torch.Tensor:
     """out[pair] = a[pair // a_div] W_e^T for the expert e whose list holds the pair; w [experts, N (gated: 2 N, gate rows
-    then up rows), K] of a's type.  gated: out = silu(gate) * up in out's type; else float32.  `tensor_cores` as the
-    routing was told."""
+    then up rows), K] of a's type.  gated: out = silu(gate) * up in out's type, or with `clamp` = (limit, alpha)
+    min(gate, limit) sigmoid(alpha min(gate, limit)) (clamp(up, -limit, limit) + 1); else float32.  `tensor_cores` as the
+    routing was told.  Pairs in no list (an expert without weights) keep what `out` held."""
+    clamped, limit, alpha = _clamp(clamp)
     _cuda(a, w, lists, counts, tiles, out)
     experts, wn, K = w.shape
     N = wn // 2 if gated else wn
     _need(a.dtype == w.dtype and a.dim() == 2 and a.shape[1] == K and a.shape[0] * a_div >= pairs, "moe_product: rows do not fit the weights")
     _need(tuple(out.shape) == (pairs, N), "moe_product: output shape does not fit")
     _check(_fn("moe", "llmx_moe_product")(_ptr(a), int(a_div), _ptr(w), _code(w), _ptr(lists), _ptr(counts), _ptr(tiles), pairs,
-                                          experts, _ptr(out), _code(out), N, K, 1 if gated else 0, 1 if tensor_cores else 0,
-                                          _stream()), "moe_product")
+                                          experts, _ptr(out), _code(out), N, K, 1 if gated else 0, clamped, limit, alpha,
+                                          1 if tensor_cores else 0, _stream()), "moe_product")
     return out
 
 
 def moe_router(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], experts: int, top: int, choice: torch.Tensor,
-               weight: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
+               weight: torch.Tensor, gate: Optional[torch.Tensor] = None, over_all: bool = False,
+               correction: Optional[torch.Tensor] = None, groups=(1, 1), scale: float = 1.0) -> None:
     """A router on the device: logits h w[:experts]^T + bias in 32-bit (w float32 [experts + extra, K]), the `top` largest to
     choice int32 [rows, top] (the lower index first among equals), the softmax over the chosen logits to weight float32
-    [rows, top]; the `extra` rows of w after the experts' give gate float32 [rows, extra] through a sigmoid."""
-    _cuda(h, w, bias, choice, weight, gate)
+    [rows, top]; the `extra` rows of w after the experts' give gate float32 [rows, extra] through a sigmoid.
+    `over_all`: s = softmax over all outputs; the choice is made by s + correction (float32 [experts] or None), of `groups` =
+    (count, keep) equal groups of neighbours only members of the `keep` with the largest best choice score; the weights are the
+    chosen s over (their sum + 1e-20), times `scale`."""
+    _cuda(h, w, bias, choice, weight, gate, correction)
+    _need(correction is None or (correction.dtype == torch.float32 and correction.numel() == experts), "moe_router: float32 correction [experts]")
+    count, keep = (int(g) for g in groups)
+    _need(over_all or (correction is None and (count, keep) == (1, 1) and scale == 1.0), "moe_router: correction, groups and scale come with over_all")
     rows, K = h.shape
     extra = w.shape[0] - experts
     _need(w.dtype == torch.float32 and w.dim() == 2 and w.shape[1] == K and extra >= 0, "moe_router: float32 weights [experts + extra, K]")
@@ -890,18 +960,28 @@ def moe_router(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], e
     _need(choice.dtype == torch.int32 and tuple(choice.shape) == (rows, top) and weight.dtype == torch.float32
           and tuple(weight.shape) == (rows, top), "moe_router: choice int32 and weight float32 [rows, top]")
     _need(extra == 0 or (gate is not None and gate.dtype == torch.float32 and gate.numel() == rows * extra), "moe_router: gate float32 [rows, extra]")
-    _check(_fn("moe", "llmx_moe_router")(_ptr(h), _code(h), _ptr(w), _ptr(bias), rows, K, experts, top, extra, _ptr(choice), _ptr(weight),
+    _check(_fn("moe", "llmx_moe_router")(_ptr(h), _code(h), _ptr(w), _ptr(bias), rows, K, experts, top, extra,
+                                         1 if over_all else 0, _ptr(correction), count, keep, float(scale), _ptr(choice), _ptr(weight),
                                          _ptr(gate), _stream()), "moe_router")
 
 
-def moe_combine_weighted_(x: torch.Tensor, y: torch.Tensor, pair_weight: torch.Tensor, top: int, factor: float = 1.0) -> torch.Tensor:
-    """x[row] += factor * sum_k pair_weight[row, k] * y[row * top + k], k in increasing order; float32."""
-    _cuda(x, y, pair_weight)
+def moe_combine_weighted_(x: torch.Tensor, y: torch.Tensor, pair_weight: torch.Tensor, top: int, factor: float = 1.0,
+                          choice: Optional[torch.Tensor] = None, experts: int = 0, h: Optional[torch.Tensor] = None,
+                          shared: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x[row] += factor * sum_k pair_weight[row, k] * y[row * top + k], k in increasing order; float32.  `choice` int32
+    [rows, top] with `experts` and `h` [rows, width]: a pair whose choice is not below `experts` takes the row's h in y's place.
+    `shared` [rows, width] and `shared_gate` [rows]: + shared_gate[row] * shared[row]."""
+    _cuda(x, y, pair_weight, choice, h, shared, shared_gate)
     rows, width = x.shape
+    _need((choice is None) == (h is None) and (choice is None or (choice.dtype == torch.int32 and choice.numel() == rows * top
+          and tuple(h.shape) == (rows, width))), "moe_combine: int32 choices and the rows' inputs come together")
+    _need((shared is None) == (shared_gate is None) and (shared is None or (shared.dtype == torch.float32 and tuple(shared.shape) == (rows, width)
+          and shared_gate.dtype == torch.float32 and shared_gate.numel() == rows)), "moe_combine: the shared part and its gate, float32")
     _need(x.dtype == torch.float32 and y.dtype == torch.float32 and tuple(y.shape) == (rows * top, width)
           and pair_weight.dtype == torch.float32 and pair_weight.numel() == rows * top, "moe_combine: shapes do not fit")
-    _check(_fn("moe", "llmx_moe_combine_weighted")(_ptr(y), _ptr(x), _ptr(pair_weight), rows, top, width, float(factor), _stream()),
-           "moe_combine_weighted")
+    _check(_fn("moe", "llmx_moe_combine_weighted")(_ptr(y), _ptr(x), _ptr(pair_weight), _ptr(choice), int(experts), _ptr(h),
+                                                   F32 if h is None else _code(h), _ptr(shared), _ptr(shared_gate), rows, top, width,
+                                                   float(factor), _stream()), "moe_combine_weighted")
     return x
 
 

@@ -4,7 +4,7 @@ from .linear import Linear
 from .norm import GroupedRMSNorm, LayerNorm, RMSNorm
 from .rope import NoPositionEncoding, RotaryEmbedding
 from .attention import Attention
-from .mlp import ClampedGLU, GatedMLP, RoutedExperts, TableRoutedExperts
+from .mlp import ActivatedMLP, ClampedGLU, GatedMLP, RoutedExperts, TableRoutedExperts
 from .block import InputFilter, ParallelBlock, PreNormBlock, SandwichBlock
 from .linear_attention import DecayedLinearAttention
 from .delta_rule import GatedDeltaRule
@@ -18,4 +18,4 @@ __all__ = ["GroupView", "Part", "Precision", "StepBatch", "Linear", "RMSNorm", "
            "RotaryEmbedding", "Attention", "GatedMLP", "PreNormBlock", "LogitsHead", "TokenEmbedding", "LayerNorm", "ClampedGLU",
            "ParallelBlock", "DecayedLinearAttention", "GatedDeltaRule", "LatentAttention",
            "TableRoutedExperts", "SelectiveStateSpace", "MaskedAttention", "MixerPair", "SandwichBlock",
-           "GroupedRMSNorm", "RoutedExperts", "InputFilter", "PairHashEmbedding"]
+           "GroupedRMSNorm", "RoutedExperts", "InputFilter", "PairHashEmbedding", "ActivatedMLP"]

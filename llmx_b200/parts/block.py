@@ -1,5 +1,5 @@
 """How a layer's parts are arranged.  PreNormBlock: x += mixer(norm(x)); x += ffn(norm(x)).
-ParallelBlock: x += mixer(norm(x)) + ffn(norm(x)).  SandwichBlock: a norm before and after each sublayer and a factor
+ParallelBlock: x += mixer(norm(x)) + ffn(norm(x)), with one norm or one for each.  SandwichBlock: a norm before and after each sublayer and a factor
 on what enters the stream: x += m * norm_b(mixer(norm_a(x))); x += m * norm_d(ffn(norm_c(x))).
 
 The names of the four parts (the prefixes of their tensors) are arguments, so
@@ -105,12 +105,17 @@ class ParallelBlock(Part):
     into the stream.  `input_filter`: the mixer reads h + filter(h) instead of h = norm(x), a causal filter over the
     request's rows on each channel (the feed-forward reads h as it is); the norm must offer `forward_filtered`, and the
     block's cache need is then the mixer's entries and, last, a state entry of (taps - 1) * width floats (the last
-    normed rows of the request; none for a filter of one tap)."""
+    normed rows of the request; none for a filter of one tap).
+
+    `ffn_norm`: the feed-forward reads a norm of its own, ffn(ffn_norm(x)), of the same x the mixer's norm reads; two norms
+    that can share a launch (`norm.pairs_with(ffn_norm)`) do.  `ffn_norm_name`: the prefix of its tensors."""
 
     def __init__(self, norm: Part, mixer: Part, ffn: Optional[Part], names=("norm", "mixer", "mlp", "filter"), factor: float = 1.0,
-                 input_filter: Optional[InputFilter] = None):
-        self.norm, self.mixer, self.ffn = norm, mixer, ffn
-        self.names = tuple(names)
+                 input_filter: Optional[InputFilter] = None, ffn_norm: Optional[Part] = None, ffn_norm_name: str = "norm2"):
+        if ffn_norm is not None and ffn is None:
+            raise ValueError("parallel block: a norm for the feed-forward needs a feed-forward")
+        self.norm, self.mixer, self.ffn, self.ffn_norm = norm, mixer, ffn, ffn_norm
+        self.names, self.ffn_norm_name = tuple(names), ffn_norm_name
         self.factor, self.input_filter = float(factor), input_filter
         if input_filter is not None and (len(self.names) < 4 or not hasattr(norm, "forward_filtered")):
             raise ValueError("parallel block: an input filter needs a name and a norm that can apply it")
@@ -120,6 +125,8 @@ class ParallelBlock(Part):
         out = {self.names[0]: self.norm, self.names[1]: self.mixer}
         if self.ffn is not None:
             out[self.names[2]] = self.ffn
+        if self.ffn_norm is not None:
+            out[self.ffn_norm_name] = self.ffn_norm
         if self.input_filter is not None:
             out[self.names[3]] = self.input_filter
         return out
@@ -161,8 +168,12 @@ class ParallelBlock(Part):
                 write_cache = True if not writes else writes[0] if len(writes) == 1 else writes
                 state = step.state(filter_entry)
             h, hm = self.norm.forward_filtered(x, self.input_filter.weight, state, step, zero=flat)
+        elif self.ffn_norm is not None and hasattr(self.norm, "pairs_with") and self.norm.pairs_with(self.ffn_norm):
+            hm, h = self.norm.forward_pair(x, self.ffn_norm, zero=flat)
         else:
             h = hm = self.norm.forward(x, zero=flat)
+            if self.ffn_norm is not None:
+                h = self.ffn_norm.forward(x)
         for z in others:
             if z is not None:
                 z.zero_()

@@ -14,13 +14,20 @@ from .linear import Linear, bare_step
 
 class TokenEmbedding(Part):
     """x[r, :] = table[ids[r], :] widened to 32-bit (src/model/arch/blocks.hpp:95-97), times `scale` when the
-    architecture has a factor on its embedding (the product is made in 32-bit).  `role`: the table's tensor role."""
+    architecture has a factor on its embedding (the product is made in 32-bit).  `role`: the table's tensor role.
+    `norm`: an RMS norm every row passes before the first layer (32-bit in and out; its tensors under `norm_name`);
+    gather, factor and norm are then one kernel."""
 
-    def __init__(self, vocab: int, hidden: int, scale: float = 1.0, role: str = "weight"):
+    def __init__(self, vocab: int, hidden: int, scale: float = 1.0, role: str = "weight", norm: Optional[Part] = None,
+                 norm_name: str = "norm"):
         self.vocab, self.hidden = int(vocab), int(hidden)
         self.scale, self.role = float(scale), role
+        self.norm, self.norm_name = norm, norm_name
         self.table: Optional[torch.Tensor] = None
         self._native: Optional[NativeHandle] = None
+
+    def children(self) -> Dict[str, Part]:
+        return {} if self.norm is None else {self.norm_name: self.norm}
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         return {self.role: TensorSpec((self.vocab, self.hidden), "table")}
@@ -32,8 +39,8 @@ class TokenEmbedding(Part):
 
     @property
     def native(self):
-        if self.scale != 1.0:
-            return None               # the runtime's embedding has no factor: the kernel with one is called from here
+        if self.scale != 1.0 or self.norm is not None:
+            return None               # the runtime's embedding has no factor and no norm: the kernels with them are called from here
         if self._native is None:
             runtime.need("rowwise")
             self._native = NativeHandle(runtime.lib().llmx_embedding_create(self.table.data_ptr(), runtime.code(self.table.dtype),
@@ -44,6 +51,9 @@ class TokenEmbedding(Part):
         if not (ids.is_cuda and ids.dtype is torch.int32 and ids.is_contiguous()):
             raise runtime.KernelError("embed: ids must be int32 on the device")
         x = torch.empty((ids.numel(), self.hidden), dtype=torch.float32, device=ids.device)
+        if self.norm is not None:
+            from .. import ops
+            return ops.embed_norm(self.table, ids, x, self.scale, self.norm.weight, self.norm.eps)
         if self.scale != 1.0:
             from .. import ops
             return ops.embed_scaled(self.table, ids, x, self.scale)

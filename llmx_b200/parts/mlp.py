@@ -105,6 +105,41 @@ class ClampedGLU(Part):
         self.down(act, out=residual, accumulate=True)
 
 
+class ActivatedMLP(Part):
+    """residual += act(h Wu^T) Wd^T, a feed-forward of two matrices.  `activation`: "relu2", the square of relu, in 32-bit.
+    `names`: the roles of the up and down weights."""
+
+    def __init__(self, hidden: int, intermediate: int, activation: str = "relu2", names=("up", "down")):
+        if activation != "relu2":
+            raise ValueError(f"activation {activation!r} has no kernel here (relu2)")
+        self.hidden, self.intermediate, self.activation, self.names = int(hidden), int(intermediate), activation, tuple(names)
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        u, d = self.names
+        return {u: TensorSpec((self.intermediate, self.hidden)), d: TensorSpec((self.hidden, self.intermediate))}
+
+    def stored_products(self):
+        return (self.up,)
+
+    def load(self, tensors, precision: Precision) -> None:
+        super().load(tensors, precision)
+        self.cleared_outputs = {}
+        u, d = self.names
+        self.up = Linear(tensors[u], precision)
+        self.down = Linear(tensors[d], precision)
+
+    def forward(self, h: torch.Tensor, step: Optional[StepBatch], residual: torch.Tensor) -> None:
+        from .. import ops
+        rows = h.shape[0]
+        if not (h.is_cuda and h.is_contiguous() and h.dtype is self.precision.act and tuple(h.shape) == (rows, self.hidden)
+                and residual.dtype is torch.float32 and residual.is_contiguous() and tuple(residual.shape) == (rows, self.hidden)):
+            raise runtime.KernelError("feed-forward: rows of the path's type and the part's width, a float32 residual")
+        up = stored_product(self, self.up, h)
+        act = torch.empty((rows, self.intermediate), dtype=self.precision.act, device=h.device)
+        ops.relu_squared(up, act)
+        self.down(act, out=residual, accumulate=True)
+
+
 class TableRoutedExperts(Part):
     """A mixture of experts without a router: an integer table [vocab, top] gives each token id its `top` experts
     (the entries of a row differ), each weighing 1 / top.
@@ -184,15 +219,35 @@ class RoutedExperts(Part):
     product).  The experts' weights are stacked as `TableRoutedExperts` stacks them and the same kernels run the
     products (csrc/moe.cu); the router writes its choice as a table [rows, top] on the device, so nothing of the routing
     is read on the host.  Tensor roles: `router`, `router.b`, `e<i>.gate|up|down`; the shared part's under `shared.`,
-    its gate `shared.sg`."""
+    its gate `shared.sg`.
+
+    Options for designs that vary it:
+        scores "all"       s = softmax over all of the router's outputs; the choice is made by s + correction (a vector
+                           under `correction_role`, or none), the weights are the chosen s over their sum (+ 1e-20)
+        groups (n, keep)   the outputs form n equal groups of neighbours; only members of the `keep` groups with the
+                           largest best choice score can be chosen (with scores "all")
+        identity           so many more outputs of the router after the experts' whose expert gives its input back
+        weight_scale       a factor on the weights
+        clamp (limit, alpha)   the experts are clamped gated units (see ClampedGLU) instead of silu(gate) * up"""
 
     few_pairs = 64
 
     def __init__(self, hidden: int, experts: int, top: int, intermediate: int, shared: Optional[Part] = None, shared_gate: bool = False,
                  names=("gate", "up", "down"), router_role: str = "router", router_bias_role: Optional[str] = "router.b",
-                 shared_name: str = "shared", shared_gate_role: str = "sg"):
-        if not 1 <= top <= experts:
+                 shared_name: str = "shared", shared_gate_role: str = "sg", scores: str = "chosen",
+                 correction_role: Optional[str] = None, groups=(1, 1), identity: int = 0, weight_scale: float = 1.0, clamp=None):
+        if scores not in ("chosen", "all"):
+            raise ValueError("experts: scores are the softmax over the chosen logits or over all")
+        if scores == "chosen" and (correction_role is not None or tuple(groups) != (1, 1) or weight_scale != 1.0):
+            raise ValueError("experts: a correction, groups and a factor on the weights come with scores over all outputs")
+        self.outputs = int(experts) + int(identity)
+        self.group_count, self.group_keep = (int(g) for g in groups)
+        if self.outputs % self.group_count or not 1 <= self.group_keep <= self.group_count:
+            raise ValueError("experts: the groups must divide the router's outputs, and some of them are kept")
+        if not 1 <= top <= self.group_keep * (self.outputs // self.group_count):
             raise ValueError("experts: a token uses between one and all of the experts")
+        self.scores, self.correction_role, self.identity = scores, correction_role, int(identity)
+        self.weight_scale, self.clamp = float(weight_scale), None if clamp is None else (float(clamp[0]), float(clamp[1]))
         self.hidden, self.experts, self.top, self.intermediate = int(hidden), int(experts), int(top), int(intermediate)
         self.shared, self.shared_gate, self.names = shared, bool(shared_gate) and shared is not None, tuple(names)
         self.router_role, self.router_bias_role, self.shared_name = router_role, router_bias_role, shared_name
@@ -204,9 +259,11 @@ class RoutedExperts(Part):
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         g, u, d = self.names
-        specs = {self.router_role: TensorSpec((self.experts, self.hidden), std=0.5)}
+        specs = {self.router_role: TensorSpec((self.outputs, self.hidden), std=0.5)}
         if self.router_bias_role is not None:
-            specs[self.router_bias_role] = TensorSpec((self.experts,), "vector", init="normal", std=0.5)
+            specs[self.router_bias_role] = TensorSpec((self.outputs,), "vector", init="normal", std=0.5)
+        if self.correction_role is not None:
+            specs[self.correction_role] = TensorSpec((self.outputs,), "vector", init="normal", std=0.1)
         if self.shared_gate:
             specs[self.gate_role] = TensorSpec((1, self.hidden), std=0.1)
         for e in range(self.experts):
@@ -214,6 +271,14 @@ class RoutedExperts(Part):
             specs[f"e{e}.{u}"] = TensorSpec((self.intermediate, self.hidden))
             specs[f"e{e}.{d}"] = TensorSpec((self.hidden, self.intermediate))
         return specs
+
+    def stored_products(self):
+        """The shared part's products whose result is stored: the block may clear their outputs in passing."""
+        return getattr(self.shared, "stored_products", tuple)()
+
+    @property
+    def cleared_outputs(self):
+        return self.shared.cleared_outputs
 
     def cleared_scratch(self, rows: int) -> int:
         """Floats of cleared scratch a step of `rows` rows needs (the gated shared part's output)."""
@@ -225,6 +290,7 @@ class RoutedExperts(Part):
         rows = [tensors[self.router_role]] + ([tensors[self.gate_role].reshape(1, self.hidden)] if self.shared_gate else [])
         self.router_w = torch.cat([r.to(torch.float32) for r in rows], dim=0).contiguous()
         self.router_b = tensors[self.router_bias_role].to(torch.float32).contiguous() if self.router_bias_role is not None else None
+        self.correction = tensors[self.correction_role].to(torch.float32).contiguous() if self.correction_role is not None else None
         act = precision.act
         self.w_gate_up = torch.stack([torch.cat([tensors[f"e{e}.{g}"], tensors[f"e{e}.{u}"]], dim=0) for e in range(self.experts)]).to(act).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.{d}"] for e in range(self.experts)]).to(act).contiguous()
@@ -242,12 +308,13 @@ class RoutedExperts(Part):
         choice = torch.empty((rows, self.top), dtype=torch.int32, device=dev)
         weight = torch.empty((rows, self.top), dtype=torch.float32, device=dev)
         gate = torch.empty((rows,), dtype=torch.float32, device=dev) if self.shared_gate else None
-        ops.moe_router(h, self.router_w, self.router_b, self.experts, self.top, choice, weight, gate)
+        ops.moe_router(h, self.router_w, self.router_b, self.outputs, self.top, choice, weight, gate, over_all=self.scores == "all",
+                       correction=self.correction, groups=(self.group_count, self.group_keep), scale=self.weight_scale)
         act = torch.empty((pairs, self.intermediate), dtype=self.precision.act, device=dev)
         y = torch.empty((pairs, self.hidden), dtype=torch.float32, device=dev)
         if self.tensor_cores and pairs <= self.few_pairs:
             # A few pairs (decoding): the experts' weights streamed once a pair; which form runs follows the step's rows alone.
-            ops.moe_product_few(h, self.top, self.w_gate_up, None, choice, pairs, act, gated=True)
+            ops.moe_product_few(h, self.top, self.w_gate_up, None, choice, pairs, act, gated=True, clamp=self.clamp)
             ops.moe_product_few(act, 1, self.w_down, None, choice, pairs, y, gated=False)
         else:
             lists = torch.empty((self.experts, pairs), dtype=torch.int32, device=dev)
@@ -255,17 +322,17 @@ class RoutedExperts(Part):
             tiles = torch.empty((ops.moe_tiles_len(pairs, self.experts),), dtype=torch.int32, device=dev)
             tc = self.tensor_cores
             ops.moe_route(None, choice, self.experts, lists, counts, tiles, tensor_cores=tc)
-            ops.moe_product(h, self.top, self.w_gate_up, lists, counts, tiles, pairs, act, gated=True, tensor_cores=tc)
+            ops.moe_product(h, self.top, self.w_gate_up, lists, counts, tiles, pairs, act, gated=True, tensor_cores=tc, clamp=self.clamp)
             ops.moe_product(act, 1, self.w_down, lists, counts, tiles, pairs, y, gated=False, tensor_cores=tc)
-        ops.moe_combine_weighted_(residual, y, weight, self.top)
-        if self.shared is None:
-            return
-        if not self.shared_gate:
+        shared_out = None
+        if self.shared_gate:
+            scratch, self.scratch = self.scratch, None
+            if scratch is None or scratch.numel() < rows * self.hidden:
+                scratch = torch.zeros(rows * self.hidden, dtype=torch.float32, device=dev)
+            shared_out = scratch[:rows * self.hidden].view(rows, self.hidden)
+            self.shared.forward(h, step, shared_out)
+        # The weighted sum, the identity experts' share of the input and the gated shared unit join the stream in one pass.
+        ops.moe_combine_weighted_(residual, y, weight, self.top, choice=choice if self.identity else None, experts=self.experts,
+                                  h=h if self.identity else None, shared=shared_out, shared_gate=gate)
+        if self.shared is not None and not self.shared_gate:
             self.shared.forward(h, step, residual)
-            return
-        scratch, self.scratch = self.scratch, None
-        if scratch is None or scratch.numel() < rows * self.hidden:
-            scratch = torch.zeros(rows * self.hidden, dtype=torch.float32, device=dev)
-        out = scratch[:rows * self.hidden].view(rows, self.hidden)
-        self.shared.forward(h, step, out)
-        ops.add_rows_(residual, out, 1.0, gate)

@@ -64,6 +64,22 @@ class RMSNorm(Part):
                                                       0 if zero is None else zero.numel()), "rmsnorm")
         return out
 
+    def forward_pair(self, x: torch.Tensor, other: "RMSNorm", zero: Optional[torch.Tensor] = None):
+        """(this norm of x, `other`'s norm of the same x) in one launch that reads x once: two RMS norms with one epsilon
+        differ in their weights alone.  `zero` as in `forward`."""
+        from .. import ops
+        if not self.pairs_with(other):
+            raise runtime.KernelError("rmsnorm pair: two RMS norms of one width and one epsilon")
+        both = torch.empty((2, x.shape[0], self.width), dtype=self.precision.act, device=x.device)
+        if zero is not None and (zero.numel() % 4 or zero.data_ptr() % 16):
+            zero.zero_()
+            zero = None
+        ops.rmsnorm_pair(x, self.weight, other.weight, self.eps, both[0], both[1], zero=zero)
+        return both[0], both[1]
+
+    def pairs_with(self, other: Part) -> bool:
+        return type(other) is RMSNorm and other.width == self.width and other.eps == self.eps
+
 
 class GroupedRMSNorm(Part):
     """RMS norm in groups: the row is split into `groups` equal consecutive parts, each divided by its own

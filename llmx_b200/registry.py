@@ -95,3 +95,4 @@ def _ensure_builtin() -> None:
     from .models import kisepel as _kisepel  # noqa: F401
     from .models import zamizen as _zamizen  # noqa: F401
     from .models import nomutar as _nomutar  # noqa: F401
+    from .models import fipadra as _fipadra  # noqa: F401
