@@ -24,7 +24,8 @@
 //             tiles; this keeps every SM streaming weights whatever N is.
 // A third form, DUAL, computes two products that share the token tile -- rows n and n + N/2 of
 // the weight (gate and up of a gated feed-forward) -- into two accumulators and writes
-// silu(gate) * up as bfloat16, so the [tokens, 2 * intermediate] float32 matrix never exists.
+// silu(gate) * up (or another gated unit, gemm_act_epilogue.cuh) as bfloat16, so the [tokens, 2 * intermediate] float32
+// matrix never exists; whole tiles may also pass one product's result through an activation (MODE_ACT).
 // A fourth form, HEADS, is the q/k/v product of an attention layer with heads of 128: the operands
 // change sides (128 tokens on the instruction's M side, 128 or 256 weight rows = one or two whole heads on
 // the narrow side), so that a thread of the epilogue holds whole heads of one token.  It norms and rotates
@@ -34,6 +35,7 @@
 // The reference has no tensor-core path for this product (its kernels: f32.gpu:1034-1084).
 #include "tc_common.cuh"
 #include "gemm_heads_epilogue.cuh"
+#include "gemm_act_epilogue.cuh"
 #include <math.h>
 
 namespace {
@@ -48,7 +50,7 @@ constexpr int EPI_WARPS = 4;
 constexpr int HEADS_TOKEN_FIRST_TILES = 16;
 constexpr int THREADS = 64 + EPI_WARPS * 32;
 
-enum : int { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_ATOMIC = 2, MODE_SWIGLU = 3 };
+enum : int { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_ATOMIC = 2, MODE_ACT = 3 };
 enum : int { ERR_PRODUCER = 101, ERR_MMA_FULL = 102, ERR_MMA_ACC = 103, ERR_EPILOGUE = 104 };
 
 template <int BN, bool DUAL>
@@ -143,7 +145,7 @@ template <int BN, bool STREAMK, bool DUAL, bool HEADS>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                void* __restrict__ C_, int M, int N, int K, int mode, int splits, int skew, int* error_word,
-               const HeadsEpilogue hp) {
+               const HeadsEpilogue hp, const ActEpilogue ae) {
     // HEADS: `map_w` is the tokens' map and N their number, `map_a` the weight's and M its rows.
     using cfg = Cfg<BN, DUAL>;
     extern __shared__ uint8_t smem_raw[];
@@ -320,15 +322,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         else tc::tmem_ld_32x16(taddr + BN + c, u);
                         tc::tmem_wait_ld();
                         if (n < N) {
-                            // silu(g) * u in float32 with the fast exponential and reciprocal (a few units in the
-                            // last place, far below the bfloat16 rounding that follows): with short inner widths
-                            // this epilogue, not the products, sets the kernel's time.
                             __nv_bfloat16* C = (__nv_bfloat16*)C_ + (size_t)(w.mt * BN + c) * N + n;
                             const int m_left = M - (w.mt * BN + c);
 #pragma unroll
                             for (int j = 0; j < CH; ++j) {
-                                const float g = __uint_as_float(r[j]), up = __uint_as_float(u[j]);
-                                const float act = __fdividef(g, 1.0f + __expf(-g)) * up;
+                                const float act = act_gated(ae, __uint_as_float(r[j]), __uint_as_float(u[j]));
                                 if (j < m_left) C[(size_t)j * N] = __float2bfloat16_rn(act);
                             }
                         }
@@ -337,7 +335,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         if (n < N) {
                             float* C = (float*)C_ + (size_t)(w.mt * BN + c) * N + n;
                             const int m_left = M - (w.mt * BN + c);        // rows of this chunk inside the matrix
-                            if (atomic) {
+                            if (!STREAMK && mode == MODE_ACT) {
+                                __nv_bfloat16* H = (__nv_bfloat16*)C_ + (size_t)(w.mt * BN + c) * N + n;
+#pragma unroll
+                                for (int j = 0; j < CH; ++j)
+                                    if (j < m_left) H[(size_t)j * N] = __float2bfloat16_rn(act_single(__uint_as_float(r[j])));
+                            } else if (atomic) {
 #pragma unroll
                                 for (int j = 0; j < CH; ++j)
                                     if (j < m_left) atomicAdd(C + (size_t)j * N, __uint_as_float(r[j]));
@@ -368,7 +371,7 @@ int g_sm_count = 0;
 
 template <int BN, bool STREAMK, bool DUAL>
 int launch(const CUtensorMap& map_w, const void* A, void* C, int M, int N, int K, int mode, int splits,
-           int* error_word, cudaStream_t stream) {
+           int* error_word, cudaStream_t stream, const ActEpilogue& ae = ActEpilogue{}) {
     using cfg = Cfg<BN, DUAL>;
     static bool configured = false;
     if (!configured) {
@@ -405,7 +408,7 @@ int launch(const CUtensorMap& map_w, const void* A, void* C, int M, int N, int K
         if (stream_ns >= STAGGER_NS) skew = (int)(100.0 * STAGGER_NS / (2 * stream_ns) + 0.5);
     }
     launch_kernel(gemm_tc_kernel<BN, STREAMK, DUAL, false>, dim3((unsigned)grid), dim3(THREADS), cfg::SMEM_BYTES, stream, 
-        map_w, map_a, C, M, N, K, mode, splits, skew, error_word, HeadsEpilogue{});
+        map_w, map_a, C, M, N, K, mode, splits, skew, error_word, HeadsEpilogue{}, ae);
     return launch_status();
 }
 
@@ -426,7 +429,7 @@ int launch_heads(const CUtensorMap& map_weight, const void* A, int tokens, int f
     long long grid = (long long)((tokens + BM - 1) / BM) * ((features + BN - 1) / BN);
     if (grid > g_sm_count) grid = g_sm_count;
     launch_kernel(gemm_tc_kernel<BN, false, false, true>, dim3((unsigned)grid), dim3(THREADS), cfg::SMEM_BYTES, stream,
-        map_tokens, map_weight, (void*)nullptr, features, tokens, K, (int)MODE_STORE, 1, 0, error_word, hp);
+        map_tokens, map_weight, (void*)nullptr, features, tokens, K, (int)MODE_STORE, 1, 0, error_word, hp, ActEpilogue{});
     return launch_status();
 }
 
@@ -521,20 +524,39 @@ LLMX_EXPORT int llmx_gemm_tc(const void* weight_map, const void* A, float* C, in
     }
 }
 
+// out = act(A W^T) as bfloat16 [M, N].  activation 0, 1 (gated): out[m, n] = glu(A W[n]^T, A W[n + N]^T), the weight has
+// 2 N rows (gate rows, then up rows), glu the silu unit or the clamped one of `limit` and `alpha`; 2: out[m, n] =
+// max(A W[n]^T, 0)^2.  `token_tile` as in llmx_gemm_tc (gated: at most 128).
+LLMX_EXPORT int llmx_gemm_tc_act(const void* weight_map, const void* A, void* out, int M, int N, int K, int activation, float limit,
+                                 float alpha, int token_tile, int* error_word, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return 0;
+    if (K <= 0 || K % 8 || ((uintptr_t)A & 15) || ((uintptr_t)out & 1)) return LLMX_ERR_UNSUPPORTED;
+    if (activation < ACT_SWIGLU || activation > ACT_RELU2) return LLMX_ERR_BAD_ARGUMENT;
+    ensure_sm_count();
+    const bool gated = activation != ACT_RELU2;
+    const ActEpilogue ae = {activation, limit, alpha};
+    int bn = token_tile;
+    if (bn == 0) bn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : gated || M <= 128 ? 128 : 256;
+    const CUtensorMap& map_w = *(const CUtensorMap*)weight_map;
+    switch (bn) {
+#define LLMX_ACT(B)                                                                                                      \
+    case B:                                                                                                              \
+        return gated ? launch<B, false, true>(map_w, A, out, M, N, K, MODE_ACT, 1, error_word, stream, ae)               \
+                     : launch<B, false, false>(map_w, A, out, M, N, K, MODE_ACT, 1, error_word, stream, ae)
+        LLMX_ACT(16);
+        LLMX_ACT(32);
+        LLMX_ACT(64);
+        LLMX_ACT(128);
+#undef LLMX_ACT
+        case 256:
+            if (!gated) return launch<256, false, false>(map_w, A, out, M, N, K, MODE_ACT, 1, error_word, stream, ae);
+            return LLMX_ERR_BAD_ARGUMENT;
+        default: return LLMX_ERR_BAD_ARGUMENT;
+    }
+}
+
 // out[m, n] = silu(A W[n]^T) * (A W[n + N]^T) as bfloat16 [M, N]; the weight has 2 N rows (gate rows, then up rows).
 LLMX_EXPORT int llmx_gemm_tc_swiglu(const void* weight_map, const void* A, void* out, int M, int N, int K,
                                     int token_tile, int* error_word, cudaStream_t stream) {
-    if (M <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 || ((uintptr_t)A & 15) || ((uintptr_t)out & 1)) return LLMX_ERR_UNSUPPORTED;
-    ensure_sm_count();
-    int bn = token_tile;
-    if (bn == 0) bn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : 128;
-    const CUtensorMap& map_w = *(const CUtensorMap*)weight_map;
-    switch (bn) {
-        case 16: return launch<16, false, true>(map_w, A, out, M, N, K, MODE_SWIGLU, 1, error_word, stream);
-        case 32: return launch<32, false, true>(map_w, A, out, M, N, K, MODE_SWIGLU, 1, error_word, stream);
-        case 64: return launch<64, false, true>(map_w, A, out, M, N, K, MODE_SWIGLU, 1, error_word, stream);
-        case 128: return launch<128, false, true>(map_w, A, out, M, N, K, MODE_SWIGLU, 1, error_word, stream);
-        default: return LLMX_ERR_BAD_ARGUMENT;
-    }
+    return llmx_gemm_tc_act(weight_map, A, out, M, N, K, ACT_SWIGLU, 0.0f, 0.0f, token_tile, error_word, stream);
 }

@@ -23,7 +23,7 @@
 //
 // Three forms share the kernel.  PLAIN: float32 output, stored or added.  DUAL: two products that share the token
 // tile -- weight rows n and n + N (gate and up of a gated feed-forward), two tiles of 128 rows a block and two
-// accumulators -- written as silu(gate) * up in bfloat16.  HEADS: the q/k/v product of heads of 128; the operands
+// accumulators -- written as silu(gate) * up (or another gated unit, gemm_act_epilogue.cuh) in bfloat16.  HEADS: the q/k/v product of heads of 128; the operands
 // change sides (the pair's 256 rows are tokens, 128 a block; the narrow side is 256 weight rows = two heads, of which
 // each block loads one), so a thread of the epilogue holds two whole heads of one token, norms and rotates them and
 // writes queries and cache rows as bfloat16 (gemm_heads_epilogue.cuh).
@@ -31,6 +31,7 @@
 // The reference has no tensor-core path for this product (its kernels: f32.gpu:1034-1084).
 #include "tc_common.cuh"
 #include "gemm_heads_epilogue.cuh"
+#include "gemm_act_epilogue.cuh"
 
 namespace {
 
@@ -39,7 +40,7 @@ constexpr int BK = 64;
 constexpr int UMMA_K = 16;
 constexpr int EPI_WARPS = 4;
 constexpr int THREADS = 64 + EPI_WARPS * 32;
-enum : int { MODE_STORE = 0, MODE_ACCUMULATE = 1 };
+enum : int { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_ACT = 2 };
 enum : int { ERR_PAIR_PRODUCER = 111, ERR_PAIR_MMA_FULL = 112, ERR_PAIR_MMA_ACC = 113, ERR_PAIR_EPILOGUE = 114 };
 
 enum : int { PLAIN = 0, DUAL = 1, HEADS = 2 };
@@ -171,7 +172,7 @@ template <int BN, int FORM>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_wide, const __grid_constant__ CUtensorMap map_narrow,
                     void* __restrict__ C_, int wide_rows, int narrow_rows, int K, int mode, int splits, int group,
-                    int tail, int* error_word, const HeadsEpilogue hp) {
+                    int tail, int* error_word, const HeadsEpilogue hp, const ActEpilogue ae) {
     using cfg = PairCfg<BN, FORM>;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -308,13 +309,11 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_wide, const __grid_c
                         tc::tmem_ld_32x32(taddr + BN + c, u);
                         tc::tmem_wait_ld();
                         if (n < N) {
-                            // silu(g) * u in float32 with the fast exponential and reciprocal, as the one-block product
                             __nv_bfloat16* out = (__nv_bfloat16*)C_ + (size_t)(w.mt * BN + c) * N + n;
                             const int m_left = M - (w.mt * BN + c);
 #pragma unroll
                             for (int j = 0; j < 32; ++j) {
-                                const float g = __uint_as_float(r[j]), up = __uint_as_float(u[j]);
-                                const float act = __fdividef(g, 1.0f + __expf(-g)) * up;
+                                const float act = act_gated(ae, __uint_as_float(r[j]), __uint_as_float(u[j]));
                                 if (j < m_left) out[(size_t)j * N] = __float2bfloat16_rn(act);
                             }
                         }
@@ -324,7 +323,12 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_wide, const __grid_c
                     if (n < N) {
                         float* out = (float*)C_ + (size_t)(w.mt * BN + c) * N + n;
                         const int m_left = M - (w.mt * BN + c);
-                        if (atomic) {
+                        if (mode == MODE_ACT) {
+                            __nv_bfloat16* half = (__nv_bfloat16*)C_ + (size_t)(w.mt * BN + c) * N + n;
+#pragma unroll
+                            for (int j = 0; j < 32; ++j)
+                                if (j < m_left) half[(size_t)j * N] = __float2bfloat16_rn(act_single(__uint_as_float(r[j])));
+                        } else if (atomic) {
 #pragma unroll
                             for (int j = 0; j < 32; ++j)
                                 if (j < m_left) atomicAdd(out + (size_t)j * N, __uint_as_float(r[j]));
@@ -364,7 +368,7 @@ void ensure_sm_count() {
 // `wide` / `narrow`: the operands' maps with boxes of 128 and BN / 2 rows; their extents in rows.
 template <int BN, int FORM>
 int launch_pair(const CUtensorMap& wide, const CUtensorMap& narrow, void* C, int wide_rows, int narrow_rows, int K, int mode,
-                int splits, const HeadsEpilogue& hp, int* error_word, cudaStream_t stream) {
+                int splits, const HeadsEpilogue& hp, int* error_word, cudaStream_t stream, const ActEpilogue& ae = ActEpilogue{}) {
     using cfg = PairCfg<BN, FORM>;
     static bool configured = false;
     if (!configured) {
@@ -413,7 +417,7 @@ int launch_pair(const CUtensorMap& wide, const CUtensorMap& narrow, void* C, int
     lc.attrs = attr;
     lc.numAttrs = llmx_pdl_enabled() ? 2 : 1;
     cudaLaunchKernelEx(&lc, gemm_tc_pair_kernel<BN, FORM>, wide, narrow, C, wide_rows, narrow_rows, K, mode, splits, group,
-                       tail, error_word, hp);
+                       tail, error_word, hp, ae);
     return launch_status();
 }
 
@@ -440,17 +444,31 @@ LLMX_EXPORT int llmx_gemm_tc_pair(const void* weight_map, const void* A, float* 
     return launch_pair<256, PLAIN>(map_w, map_a, C, N, M, K, mode, splits, HeadsEpilogue{}, error_word, stream);
 }
 
-// out[m, n] = silu(A W[n]^T) * (A W[n + N]^T) as bfloat16 [M, N] on pairs of SMs; the weight has 2 N rows (gate rows,
-// then up rows) and `weight_map` boxes of 128 rows.  A pair's tile: 256 outputs x 128 tokens.
-LLMX_EXPORT int llmx_gemm_tc_pair_swiglu(const void* weight_map, const void* A, void* out, int M, int N, int K,
-                                         int* error_word, cudaStream_t stream) {
+// out = act(A W^T) as bfloat16 [M, N] on pairs of SMs; `weight_map` with boxes of 128 rows; activations as in
+// llmx_gemm_tc_act.  A pair's tile: 256 outputs x 128 tokens (gated, the weight then has 2 N rows), or x `token_tile`
+// (128 or 256) tokens.
+LLMX_EXPORT int llmx_gemm_tc_pair_act(const void* weight_map, const void* A, void* out, int M, int N, int K, int activation,
+                                      float limit, float alpha, int token_tile, int* error_word, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)A & 15) || ((uintptr_t)out & 1)) return LLMX_ERR_UNSUPPORTED;
+    if (activation < ACT_SWIGLU || activation > ACT_RELU2) return LLMX_ERR_BAD_ARGUMENT;
+    const bool gated = activation != ACT_RELU2;
+    if (token_tile != 128 && (token_tile != 256 || gated)) return LLMX_ERR_BAD_ARGUMENT;
     ensure_sm_count();
+    const ActEpilogue ae = {activation, limit, alpha};
     const CUtensorMap& map_w = *(const CUtensorMap*)weight_map;
     CUtensorMap map_a;
-    if (int e = llmx_make_map_bf16_2d(&map_a, A, (uint64_t)M, (uint64_t)K, 64, BK)) return e;
-    return launch_pair<128, DUAL>(map_w, map_a, out, N, M, K, MODE_STORE, 1, HeadsEpilogue{}, error_word, stream);
+    if (int e = llmx_make_map_bf16_2d(&map_a, A, (uint64_t)M, (uint64_t)K, token_tile / 2, BK)) return e;
+    if (gated) return launch_pair<128, DUAL>(map_w, map_a, out, N, M, K, MODE_STORE, 1, HeadsEpilogue{}, error_word, stream, ae);
+    if (token_tile == 128) return launch_pair<128, PLAIN>(map_w, map_a, out, N, M, K, MODE_ACT, 1, HeadsEpilogue{}, error_word, stream, ae);
+    return launch_pair<256, PLAIN>(map_w, map_a, out, N, M, K, MODE_ACT, 1, HeadsEpilogue{}, error_word, stream, ae);
+}
+
+// out[m, n] = silu(A W[n]^T) * (A W[n + N]^T) as bfloat16 [M, N] on pairs of SMs; the weight has 2 N rows (gate rows,
+// then up rows).
+LLMX_EXPORT int llmx_gemm_tc_pair_swiglu(const void* weight_map, const void* A, void* out, int M, int N, int K,
+                                         int* error_word, cudaStream_t stream) {
+    return llmx_gemm_tc_pair_act(weight_map, A, out, M, N, K, ACT_SWIGLU, 0.0f, 0.0f, 128, error_word, stream);
 }
 
 // The q/k/v product of a layer whose heads are 128 wide, finished in the epilogue, on pairs of SMs: the arguments of

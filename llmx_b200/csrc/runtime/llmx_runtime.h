@@ -182,6 +182,11 @@ int llmx_embedding_forward(llmx_part*, const llmx_step*, const int* ids, float* 
 int llmx_head_forward(llmx_part*, const llmx_step*, const float* x, float* logits);
 int llmx_linear_forward(llmx_part*, const llmx_step*, const void* a, int rows, float* out, int accumulate, int cleared);
 int llmx_linear_gated(llmx_part*, const llmx_step*, const void* a, int rows, void* out);
+// The product with an activation in its epilogue, out in the path's type: 0: silu(gate) * up, 1: the clamped gated unit of
+// `limit` and `alpha` (both of a stacked gate/up weight; out is half as wide), 2: the square of relu.  For as many rows as
+// llmx_linear_fuses_activation names (with few rows the product is cut by k ranges, whose sums cannot pass through it).
+int llmx_linear_activated(llmx_part*, const llmx_step*, const void* a, int rows, void* out, int activation, float limit, float alpha);
+int llmx_linear_fuses_activation(llmx_part*, int rows);
 // Floats (a multiple of 4, or 0) a mixer or feed-forward wants zeroed before its forward for this many rows: the
 // norm in front of it clears them in passing.  The buffer itself is the caller's.
 long long llmx_part_wants_cleared(llmx_part*, const llmx_step*, int rows);

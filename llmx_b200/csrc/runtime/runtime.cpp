@@ -48,6 +48,8 @@ typedef cudaStream_t S;
     X(llmx_gemm_tc_weight_map_box, (void*, const void*, int, int, int))                                                   \
     X(llmx_gemm_tc, (const void*, const void*, float*, int, int, int, int, int, int, int, int*, S))                       \
     X(llmx_gemm_tc_pair, (const void*, const void*, float*, int, int, int, int, int, int, int*, S))                       \
+    X(llmx_gemm_tc_act, (const void*, const void*, void*, int, int, int, int, float, float, int, int*, S))                \
+    X(llmx_gemm_tc_pair_act, (const void*, const void*, void*, int, int, int, int, float, float, int, int*, S))           \
     X(llmx_gemm_tc_pair_swiglu, (const void*, const void*, void*, int, int, int, int*, S))                                \
     X(llmx_gemm_tc_pair_heads, (const void*, const void*, int, int, const float*, const float*, float, const float*,      \
                                 const float*, const int*, const int*, void*, void*, int, int, int, int*, S))              \
@@ -544,6 +546,23 @@ struct Linear : llmx_part {
         if (!invariant() && (g_pair_products & PAIR_GATED) && rows >= PAIR_MIN_ROWS)
             return CALL(c, llmx_gemm_tc_pair_swiglu, 1, (const void*)map128, a, out, rows, N / 2, K, c.s->error_word, c.stream);
         return CALL(c, llmx_gemm_tc_swiglu, 1, (const void*)map128, a, out, rows, N / 2, K, invariant() ? 128 : 0, c.s->error_word, c.stream);
+    }
+    // out = act(a W^T) in the path's type, with the activation in the product's epilogue (where `fused_gate` says so):
+    // activation 0: silu(gate) up, 1: the clamped gated unit (both of a stacked gate/up weight), 2: the square of relu.
+    int activated(Ctx& c, const void* a, int rows, void* out, int activation, float limit, float alpha) {
+        if (ensure_map(c)) return c.status;
+        const bool gated = activation != 2;
+        const int outputs = gated ? N / 2 : N;
+        if (!invariant() && (g_pair_products & PAIR_GATED) && rows >= PAIR_MIN_ROWS) {
+            // One product: tiles of 128 or 256 tokens, whichever ends sooner in whole rounds over the pairs of SMs (a wide
+            // tile takes in fewer bytes a multiply-add, so it wins a tie).
+            const int pairs = std::max(sms() / 2, 1), wide = cdiv(outputs, 256);
+            const int tile = !gated && 2 * cdiv(wide * cdiv(rows, 256), pairs) <= cdiv(wide * cdiv(rows, 128), pairs) ? 256 : 128;
+            return CALL(c, llmx_gemm_tc_pair_act, 1, (const void*)map128, a, out, rows, outputs, K, activation, limit, alpha, tile,
+                        c.s->error_word, c.stream);
+        }
+        return CALL(c, llmx_gemm_tc_act, 1, (const void*)map128, a, out, rows, outputs, K, activation, limit, alpha,
+                    invariant() || rows > 64 ? 128 : 0, c.s->error_word, c.stream);
     }
     int ensure_head_map(Ctx& c, int tile) {
         const int i = tile == 256;
@@ -1281,6 +1300,19 @@ LLMX_API int llmx_linear_gated(llmx_part* p, const llmx_step* s, const void* a, 
     if (!l || !good_step(s) || !l->tensor_core) return fail(LLMX_RT_ERR_BAD_ARGUMENT, "llmx_linear_gated: not a tensor-core linear part");
     Ctx c(s, false);
     l->gated(c, a, rows, out);
+    return finish(c);
+}
+LLMX_API int llmx_linear_fuses_activation(llmx_part* p, int rows) {
+    Linear* l = as<Linear>(p, PART_LINEAR);
+    return l && l->fused_gate(rows) ? 1 : 0;
+}
+LLMX_API int llmx_linear_activated(llmx_part* p, const llmx_step* s, const void* a, int rows, void* out, int activation, float limit,
+                                   float alpha) {
+    Linear* l = as<Linear>(p, PART_LINEAR);
+    if (!l || !good_step(s) || !l->tensor_core || activation < 0 || activation > 2)
+        return fail(LLMX_RT_ERR_BAD_ARGUMENT, "llmx_linear_activated: not a tensor-core linear part, or no such activation");
+    Ctx c(s, false);
+    l->activated(c, a, rows, out, activation, limit, alpha);
     return finish(c);
 }
 LLMX_API int llmx_linear_adds_pieces(llmx_part* p, int rows) {

@@ -14,6 +14,8 @@ _i, _p = ctypes.c_int, ctypes.c_void_p
 register_signature("gemm_tc", "llmx_gemm_tc_weight_map", [_p, _p, _i, _i])
 register_signature("gemm_tc", "llmx_gemm_tc", [_p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _p])
 register_signature("gemm_tc_pair", "llmx_gemm_tc_pair", [_p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _p])
+register_signature("gemm_tc", "llmx_gemm_tc_act", [_p, _p, _p, _i, _i, _i, _i, ctypes.c_float, ctypes.c_float, _i, _p, _p])
+register_signature("gemm_tc_pair", "llmx_gemm_tc_pair_act", [_p, _p, _p, _i, _i, _i, _i, ctypes.c_float, ctypes.c_float, _i, _p, _p])
 register_signature("gemm_tc_pair", "llmx_gemm_tc_pair_swiglu", [_p, _p, _p, _i, _i, _i, _p, _p])
 register_signature("gemm_tc_pair", "llmx_gemm_tc_pair_heads", [_p, _p, _i, _i, _p, _p, ctypes.c_float, _p, _p, _p, _p, _p, _p,
                                                                _i, _i, _i, _p, _p])
@@ -144,6 +146,24 @@ def gemm_tc_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, wmap: Op
         return out
     _check(_fn("gemm_tc", "llmx_gemm_tc_swiglu")(ctypes.c_void_p(wmap.address), _ptr(a), _ptr(out), m, f, k,
                                                  token_tile, _ptr(error_word(a.device)), _stream()), "gemm_tc_swiglu")
+    return out
+
+
+def gemm_tc_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activation: str, limit: float = 0.0, alpha: float = 0.0,
+                token_tile: int = 0, pair: bool = False) -> torch.Tensor:
+    """out = act(a @ w.T) as bfloat16, the activation in the product's epilogue: "swiglu" and "clamped_glu" over a weight of
+    gate rows, then up rows (out half as wide), "relu2" over a plain one.  `pair`: on pairs of SMs (token tile 128 or 256)."""
+    _cuda(a, w, out)
+    kind = ("swiglu", "clamped_glu", "relu2").index(activation)
+    m, k = a.shape
+    f = w.shape[0] // 2 if kind < 2 else w.shape[0]
+    _need(a.dtype is torch.bfloat16 and w.dtype is torch.bfloat16 and out.dtype is torch.bfloat16, "gemm_tc_act: bfloat16 inputs and output")
+    _need(w.shape[0] == (2 * f if kind < 2 else f) and w.shape[1] == k and tuple(out.shape) == (m, f) and k % 8 == 0,
+          "gemm_tc_act: shapes do not fit")
+    wmap = weight_map(w)
+    lib, name = ("gemm_tc_pair", "llmx_gemm_tc_pair_act") if pair else ("gemm_tc", "llmx_gemm_tc_act")
+    _check(_fn(lib, name)(ctypes.c_void_p(wmap.address), _ptr(a), _ptr(out), m, f, k, kind, float(limit), float(alpha),
+                          (token_tile or 128) if pair else token_tile, _ptr(error_word(a.device)), _stream()), name)
     return out
 
 

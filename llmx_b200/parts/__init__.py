@@ -1,6 +1,6 @@
 """Parts a model is put together from."""
 from .base import GroupView, Part, Precision, StepBatch
-from .linear import Linear
+from .linear import ActivatedLinear, Linear
 from .norm import GroupedRMSNorm, LayerNorm, RMSNorm
 from .rope import NoPositionEncoding, RotaryEmbedding
 from .attention import Attention
@@ -18,4 +18,4 @@ __all__ = ["GroupView", "Part", "Precision", "StepBatch", "Linear", "RMSNorm", "
            "RotaryEmbedding", "Attention", "GatedMLP", "PreNormBlock", "LogitsHead", "TokenEmbedding", "LayerNorm", "ClampedGLU",
            "ParallelBlock", "DecayedLinearAttention", "GatedDeltaRule", "LatentAttention",
            "TableRoutedExperts", "SelectiveStateSpace", "MaskedAttention", "MixerPair", "SandwichBlock",
-           "GroupedRMSNorm", "RoutedExperts", "InputFilter", "PairHashEmbedding", "ActivatedMLP"]
+           "GroupedRMSNorm", "RoutedExperts", "InputFilter", "PairHashEmbedding", "ActivatedMLP", "ActivatedLinear"]

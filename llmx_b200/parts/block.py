@@ -152,6 +152,7 @@ class ParallelBlock(Part):
                     wanted.append((part, lin, n))
         # A part may also ask for cleared scratch of its own (`cleared_scratch(rows)` floats, handed over as `part.scratch`).
         scratch = [(p, (p.cleared_scratch(rows) + 3) & ~3) for p in (self.mixer, self.ffn) if p is not None and hasattr(p, "cleared_scratch")]
+        scratch = [(p, n) for p, n in scratch if n]
         gathered = ((rows * x.shape[1] + 3) & ~3) if self.gathered else 0
         total = gathered + sum(n for _, _, n in wanted) + sum(n for _, n in scratch)
         flat = torch.empty(total, dtype=torch.float32, device=x.device) if total else None

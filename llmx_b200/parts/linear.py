@@ -98,9 +98,49 @@ class Linear:
         must start from zeros when the product is to be stored."""
         return bool(runtime.lib().llmx_linear_adds_pieces(self.native, int(rows)))
 
+    def fuses_activation(self, rows: int) -> bool:
+        """Whether an activation can be applied in this product's epilogue for this many rows."""
+        return self.tensor_core and bool(runtime.lib().llmx_linear_fuses_activation(self.native, int(rows)))
+
     def output_to_clear(self, rows: int, device) -> Optional[torch.Tensor]:
         """A fresh output for `rows` rows if the product wants it cleared by whoever runs before it
         (then pass it back with `cleared=True`), else None."""
         if not self.adds_pieces(rows) or (rows * self.out_features) % 4:
             return None
         return torch.empty((rows, self.out_features), dtype=torch.float32, device=device)
+
+
+class ActivatedLinear(Linear):
+    """A product whose result passes an activation and is kept in the path's type: `activation` is ("clamped_glu", limit,
+    alpha) over a stacked gate/up weight (the output is half as wide) or ("relu2",).  With many rows the activation is the
+    product's epilogue; with few (the product is then cut by k ranges, whose partial sums cannot pass through it), on the
+    float32 path and for widths the tensor-core product does not take, it is a kernel after the product."""
+
+    _KINDS = {"clamped_glu": 1, "relu2": 2}
+
+    def __init__(self, weight: torch.Tensor, precision: Precision, activation):
+        super().__init__(weight, precision)
+        self.kind, self.limit, self.alpha = (tuple(activation) + (0.0, 0.0))[:3]
+        if self.kind not in self._KINDS:
+            raise ValueError(f"activation {self.kind!r} has no kernel here ({', '.join(self._KINDS)})")
+        self.outputs = self.out_features // 2 if self.kind == "clamped_glu" else self.out_features
+
+    def adds_pieces(self, rows: int) -> bool:
+        return not self.fuses_activation(rows) and super().adds_pieces(rows)
+
+    def activated(self, part, a: torch.Tensor) -> torch.Tensor:
+        """act(a @ W.T) [rows, outputs] of the path's type; `part`: the part that holds the product (see `stored_product`)."""
+        from .. import ops
+        rows = a.shape[0]
+        act = torch.empty((rows, self.outputs), dtype=self.precision.act, device=a.device)
+        if self.fuses_activation(rows):
+            if not (a.is_cuda and a.is_contiguous() and a.dtype is self.weight.dtype and a.shape[1] == self.in_features):
+                raise runtime.KernelError("linear: rows of the weight's type and input width")
+            s = bare_step(a.device)
+            runtime.check(runtime.lib().llmx_linear_activated(self.native, ctypes.byref(s), a.data_ptr(), rows, act.data_ptr(),
+                                                              self._KINDS[self.kind], float(self.limit), float(self.alpha)), "linear")
+            return act
+        product = stored_product(part, self, a)
+        if self.kind == "clamped_glu":
+            return ops.clamped_glu(product, act, self.limit, self.alpha)
+        return ops.relu_squared(product, act)

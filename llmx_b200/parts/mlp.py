@@ -14,7 +14,7 @@ import torch
 from .. import runtime
 from ..weights.spec import TensorSpec
 from .base import NativeHandle, Part, Precision, StepBatch
-from .linear import Linear, call_struct, stored_product
+from .linear import ActivatedLinear, Linear, call_struct
 
 
 class GatedMLP(Part):
@@ -71,8 +71,8 @@ class ClampedGLU(Part):
     """residual += (g sigmoid(alpha g) (u + 1)) Wd^T with g = min(h Wg^T, limit), u = clamp(h Wu^T, -limit, limit).
 
     The gate is cut from above only, the linear branch on both sides and shifted by one; `limit` and `alpha` are
-    arguments.  Gate and up weights are stacked so one product gives both; the activation is `llmx_clamped_glu`
-    (csrc/rowwise.cu) in 32-bit.  `names`: the three tensors' roles."""
+    arguments.  Gate and up weights are stacked so one product gives both; the activation, in 32-bit, is the product's
+    epilogue when rows are many and a kernel of its own when they are few.  `names`: the three tensors' roles."""
 
     def __init__(self, hidden: int, intermediate: int, limit: float, alpha: float = 1.702, names=("gate", "up", "down")):
         self.hidden, self.intermediate = int(hidden), int(intermediate)
@@ -90,23 +90,20 @@ class ClampedGLU(Part):
         super().load(tensors, precision)
         self.cleared_outputs = {}
         g, u, d = self.names
-        self.gate_up = Linear(torch.cat([tensors[g], tensors[u]], dim=0), precision)
+        self.gate_up = ActivatedLinear(torch.cat([tensors[g], tensors[u]], dim=0), precision, ("clamped_glu", self.limit, self.alpha))
         self.down = Linear(tensors[d], precision)
 
     def forward(self, h: torch.Tensor, step: Optional[StepBatch], residual: torch.Tensor) -> None:
-        from .. import ops
         rows = h.shape[0]
         if not (h.is_cuda and h.is_contiguous() and h.dtype is self.precision.act and tuple(h.shape) == (rows, self.hidden)
                 and residual.dtype is torch.float32 and residual.is_contiguous() and tuple(residual.shape) == (rows, self.hidden)):
             raise runtime.KernelError("feed-forward: rows of the path's type and the part's width, a float32 residual")
-        gu = stored_product(self, self.gate_up, h)
-        act = torch.empty((rows, self.intermediate), dtype=self.precision.act, device=h.device)
-        ops.clamped_glu(gu, act, self.limit, self.alpha)
-        self.down(act, out=residual, accumulate=True)
+        self.down(self.gate_up.activated(self, h), out=residual, accumulate=True)
 
 
 class ActivatedMLP(Part):
-    """residual += act(h Wu^T) Wd^T, a feed-forward of two matrices.  `activation`: "relu2", the square of relu, in 32-bit.
+    """residual += act(h Wu^T) Wd^T, a feed-forward of two matrices.  `activation`: "relu2", the square of relu, in 32-bit (the
+    product's epilogue when rows are many, a kernel of its own when they are few).
     `names`: the roles of the up and down weights."""
 
     def __init__(self, hidden: int, intermediate: int, activation: str = "relu2", names=("up", "down")):
@@ -125,19 +122,15 @@ class ActivatedMLP(Part):
         super().load(tensors, precision)
         self.cleared_outputs = {}
         u, d = self.names
-        self.up = Linear(tensors[u], precision)
+        self.up = ActivatedLinear(tensors[u], precision, (self.activation,))
         self.down = Linear(tensors[d], precision)
 
     def forward(self, h: torch.Tensor, step: Optional[StepBatch], residual: torch.Tensor) -> None:
-        from .. import ops
         rows = h.shape[0]
         if not (h.is_cuda and h.is_contiguous() and h.dtype is self.precision.act and tuple(h.shape) == (rows, self.hidden)
                 and residual.dtype is torch.float32 and residual.is_contiguous() and tuple(residual.shape) == (rows, self.hidden)):
             raise runtime.KernelError("feed-forward: rows of the path's type and the part's width, a float32 residual")
-        up = stored_product(self, self.up, h)
-        act = torch.empty((rows, self.intermediate), dtype=self.precision.act, device=h.device)
-        ops.relu_squared(up, act)
-        self.down(act, out=residual, accumulate=True)
+        self.down(self.up.activated(self, h), out=residual, accumulate=True)
 
 
 class TableRoutedExperts(Part):

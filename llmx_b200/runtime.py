@@ -111,6 +111,8 @@ _SIGNATURES = {
     "llmx_head_forward": (_i, [_p, _SP, _p, _p]),
     "llmx_linear_forward": (_i, [_p, _SP, _p, _i, _p, _i, _i]),
     "llmx_linear_gated": (_i, [_p, _SP, _p, _i, _p]),
+    "llmx_linear_activated": (_i, [_p, _SP, _p, _i, _p, _i, _f, _f]),
+    "llmx_linear_fuses_activation": (_i, [_p, _i]),
     "llmx_part_wants_cleared": (_ll, [_p, _SP, _i]),
     "llmx_linear_adds_pieces": (_i, [_p, _i]),
     "llmx_part_workspace": (_sz, [_p, _SP, _i, _i]),
@@ -130,6 +132,7 @@ KERNEL_LIBS: Dict[str, str] = {
     "llmx_gemm_plain": "gemm_plain", "llmx_attention_plain": "attention_plain",
     "llmx_gemm_tc_weight_map": "gemm_tc", "llmx_gemm_tc_weight_map_box": "gemm_tc", "llmx_gemm_tc": "gemm_tc",
     "llmx_gemm_tc_swiglu": "gemm_tc", "llmx_gemm_tc_heads": "gemm_tc", "llmx_gemm_tc_pair": "gemm_tc_pair",
+    "llmx_gemm_tc_act": "gemm_tc", "llmx_gemm_tc_pair_act": "gemm_tc_pair",
     "llmx_gemm_tc_pair_swiglu": "gemm_tc_pair", "llmx_gemm_tc_pair_heads": "gemm_tc_pair",
     "llmx_attn_cache_map": "attention_decode", "llmx_attn_decode_fused": "attention_decode",
     "llmx_attn_decode_qkv": "attention_decode", "llmx_attn_decode_max_clusters": "attention_decode",
