@@ -136,6 +136,10 @@ def reference_arm(args):
 # heads; the first layer's feed-forward dense, the others' Kisepel's experts with a router; a three-tap input filter, eight norm
 # groups, a pair table of 32,749 buckets) beside the two models that have its kernels' nearest relatives: a Zamizen whose
 # layers are all grouped-query attention (the same attention kernels, a filter, a factor on the residual) and the Kisepel.
+# `--design fipadra`: a Fipadra of as many layers (retention, latent attention under the window, the delta rule in turn; every
+# second layer's feed-forward Kisepel's experts with 4 identity experts beside them, in 5 groups of which 3 are kept, the others'
+# dense) beside the two models that have its kernels' nearest relatives: the Buzetar (the same three kinds of mixers) and the
+# Nomutar (routed experts under a gated shared unit).
 DESIGN_SIZES = {
     "w2048": dict(width=2048, heads=16, ff=6144, vocab=32768, q_rank=768, kv_rank=512, rot=64, window=2048, layers=6),
     "w4096": dict(width=4096, heads=32, ff=12288, vocab=32768, q_rank=1536, kv_rank=512, rot=64, window=4096, layers=3),
@@ -149,7 +153,7 @@ def design_bench(args) -> int:
     import statistics
     import torch
     from llmx_b200 import ops
-    from llmx_b200.config import BuzetarConfig, KisepelConfig, NomutarConfig, Qwen3Config, ZamizenConfig
+    from llmx_b200.config import BuzetarConfig, FipadraConfig, KisepelConfig, NomutarConfig, Qwen3Config, ZamizenConfig
     from llmx_b200.engine import Engine, EngineOptions, StepEntry
     from llmx_b200.engine.decode_loop import DecodeSession
     torch.cuda.set_device(0)
@@ -217,7 +221,7 @@ def design_bench(args) -> int:
             buz_latent = BuzetarConfig.from_dict({"architecture": "Buzetar", "vocab": z["vocab"], "width": E, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
                                                   "logit_scale": 1.0, "layers": [all_latent] * L})
             runs = (("zamizen", zam), ("buzetar_latent", buz_latent), ("qwen3", qwen))
-        if args.design == "nomutar":
+        if args.design in ("nomutar", "fipadra"):
             G = max(H // 4, 1)
             head = {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
             ramp = {"base": 1000000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 16.0, "slow": 2.0}}
@@ -235,6 +239,16 @@ def design_bench(args) -> int:
             zam_attention = ZamizenConfig.from_dict({"architecture": "Zamizen", "vocab": z["vocab"], "width": E, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
                                                      "layers": [{"type": "attention", "mixer": gqa, "mlp": {"kind": "dense", "ff": F}}] * L})
             runs = (("nomutar", nom), ("zamizen_attention", zam_attention), ("kisepel", kis))
+        if args.design == "fipadra":
+            fip_mixers = [
+                {"type": "retention", "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": decays, "rot": {"base": 10000.0, "dims": 128}}},
+                {"type": "latent_attention", "mixer": kinds[1]["mixer"]}, {"type": "delta", "mixer": kinds[2]["mixer"]}]
+            fip_mlps = [{"kind": "dense", "ff": F},
+                        {"kind": "moe", "expert": {"ff": F // 4, "limit": 7.0}, "shared": {"ff": F // 2, "limit": 7.0},
+                         "router": {"experts": 16, "identity": 4, "top": 2, "scale": 1.5, "groups": {"count": 5, "keep": 3}}}]
+            fip = FipadraConfig.from_dict({"architecture": "Fipadra", "vocab": z["vocab"], "width": E, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+                                           "layers": [dict(fip_mixers[i % 3], mlp=fip_mlps[i % 2]) for i in range(L)]})
+            runs = (("fipadra", fip), ("buzetar", buz), ("nomutar", nom))
         res = {"config": dict(z)}
         out["sizes"][name] = res                                # filled as the arms end, so that a run that stops early says what it has
         for tag, cfg in runs:
@@ -260,6 +274,7 @@ def design_bench(args) -> int:
             engine.end("prefill")
             pf_ms = statistics.median(times)
             r = {"prefill_tok_s": round(T * 1e3 / pf_ms, 1), "prefill_ms": round(pf_ms, 3),
+                 "prefill_calls_by_kernel": {k: v[0] for k, v in kt.by_function.items()},
                  "prefill_ms_by_kernel": {k: round(v[1], 4) for k, v in sorted(kt.by_function.items(), key=lambda kv: -kv[1][1])}}
             print(f"[bench] {name} {tag}: decode", file=sys.stderr, flush=True)
             rids = [("bench", i) for i in range(B)]
@@ -271,6 +286,7 @@ def design_bench(args) -> int:
                 engine.step([StepEntry(rid, [1], [0]) for rid in rids])
             with ops.kernel_times() as kt:
                 engine.step([StepEntry(rid, [1], [0]) for rid in rids])
+            r["decode_calls_by_kernel"] = {k: v[0] for k, v in kt.by_function.items()}
             r["decode_ms_by_kernel"] = {k: round(v[1], 4) for k, v in sorted(kt.by_function.items(), key=lambda kv: -kv[1][1])}
             session = DecodeSession(engine, rids)
             tokens = torch.randint(0, vocab, (B,), generator=host_gen).tolist()
@@ -315,10 +331,11 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true")
     ap.add_argument("--only", choices=["decode", "prefill", "sample"], default=None,
                     help="run one part only (for profiling); the line then holds only that part")
-    ap.add_argument("--design", choices=["buzetar", "kisepel", "zamizen", "nomutar"], default=None,
+    ap.add_argument("--design", choices=["buzetar", "kisepel", "zamizen", "nomutar", "fipadra"], default=None,
                     help="instead of the default workload: prompt and decode throughput of this design at sizes that resemble a "
                          "real model's layers, beside the closest other design of equal size (Buzetar beside Qwen3, Kisepel beside Buzetar, "
-                         "Zamizen beside an all-latent Buzetar and Qwen3, Nomutar beside an all-attention Zamizen and Kisepel; one JSON line of its own)")
+                         "Zamizen beside an all-latent Buzetar and Qwen3, Nomutar beside an all-attention Zamizen and Kisepel, Fipadra beside Buzetar "
+                         "and Nomutar; one JSON line of its own)")
     ap.add_argument("--design-size", default=None, help="with --design: one of " + ", ".join(sorted(DESIGN_SIZES)) + " (default: all)")
     args = ap.parse_args()
     if args.impl == "reference":

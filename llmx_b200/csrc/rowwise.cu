@@ -517,10 +517,19 @@ LLMX_EXPORT int llmx_embed_scaled(const void* table, int table_dtype, const int*
 }
 
 // ---------------------------------------------------------------------------
-// Embedding with a norm: z = table[ids[r], :] * scale; x[r, :] = z / sqrt(mean(z^2) + eps) * w, 32-bit.  One block a row;
-// the second pass finds the row in the caches.
+// Embedding with a norm: z = table[ids[r], :] * scale; x[r, :] = z / sqrt(mean(z^2) + eps) * w, 32-bit.  One block a row.
+// REGS (widths that are a multiple of 4 and at most 4 * NORM_VEC_MAX * blockDim): the row stays in registers between its
+// two passes, read in pieces of four values; else the second pass finds it in the caches.
 // ---------------------------------------------------------------------------
-template <typename T>
+__device__ __forceinline__ float4 read4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 read4(const __nv_bfloat16* p) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename T, bool REGS>
 __global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x, int width,
                                   int table_rows, float scale, const float* __restrict__ w, float eps) {
     pdl_trigger();
@@ -534,23 +543,54 @@ __global__ void embed_norm_kernel(const T* __restrict__ table, const int* __rest
     }
     const T* src = table + (size_t)id * width;
     float s = 0.0f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = to_float(src[i]) * scale;
-        s = fmaf(v, v, s);
+    if constexpr (REGS) {
+        const int n4 = width >> 2;
+        float4 v[NORM_VEC_MAX];
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            v[k] = i < n4 ? read4(src + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            v[k] = make_float4(v[k].x * scale, v[k].y * scale, v[k].z * scale, v[k].w * scale);
+            s = fmaf(v[k].x, v[k].x, s);
+            s = fmaf(v[k].y, v[k].y, s);
+            s = fmaf(v[k].z, v[k].z, s);
+            s = fmaf(v[k].w, v[k].w, s);
+        }
+        const float rr = 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps);
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < n4) {
+                const float4 ww = read4(w + 4 * i);
+                store4(dst + 4 * i, v[k].x * (rr * ww.x), v[k].y * (rr * ww.y), v[k].z * (rr * ww.z), v[k].w * (rr * ww.w));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            const float v = to_float(src[i]) * scale;
+            s = fmaf(v, v, s);
+        }
+        const float rr = 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps);
+        for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = to_float(src[i]) * scale * (rr * w[i]);
     }
-    s = block_sum(s, scratch);
-    const float rr = 1.0f / sqrtf(s / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = to_float(src[i]) * scale * (rr * w[i]);
 }
 
 LLMX_EXPORT int llmx_embed_norm(const void* table, int table_dtype, const int* ids, float* x, int rows, int width, int table_rows,
                                 float scale, const float* w, float eps, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (w == nullptr) return LLMX_ERR_BAD_ARGUMENT;
-    if (table_dtype == LLMX_BF16)
-        launch_kernel(embed_norm_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, stream, (const __nv_bfloat16*)table, ids, x, width, table_rows, scale, w, eps);
-    else
-        launch_kernel(embed_norm_kernel<float>, dim3(rows), dim3(256), 0, stream, (const float*)table, ids, x, width, table_rows, scale, w, eps);
+    if (w == nullptr || width <= 0) return LLMX_ERR_BAD_ARGUMENT;
+    const bool regs = width % 4 == 0 && width <= 4 * NORM_VEC_MAX * 256 && !(((uintptr_t)table | (uintptr_t)x | (uintptr_t)w) & 15);
+    const int threads = regs ? norm_threads(width) : 256;
+#define LLMX_EMBED(T, R) \
+    launch_kernel(embed_norm_kernel<T, R>, dim3(rows), dim3(threads), 0, stream, (const T*)table, ids, x, width, table_rows, scale, w, eps)
+    if (table_dtype == LLMX_BF16 && regs) LLMX_EMBED(__nv_bfloat16, true);
+    else if (table_dtype == LLMX_BF16) LLMX_EMBED(__nv_bfloat16, false);
+    else if (regs) LLMX_EMBED(float, true);
+    else LLMX_EMBED(float, false);
+#undef LLMX_EMBED
     return launch_status();
 }
 
