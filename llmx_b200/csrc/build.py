@@ -190,8 +190,32 @@ def load(name: str) -> ctypes.CDLL:
                 lib = ctypes.CDLL(path)
             except OSError as e:
                 raise BuildError(f"cannot load {path}: {e}") from None
+            _set_overlap_of(lib)
             _loaded[name] = lib
         return lib
+
+
+_overlap = True
+
+
+def _set_overlap_of(lib: ctypes.CDLL) -> None:
+    try:
+        ctypes.c_int.in_dll(lib, "llmx_launch_overlap").value = 1 if _overlap else 0
+    except ValueError:
+        pass                     # a library without kernels (the runtime)
+
+
+def set_overlap(on: bool) -> None:
+    """Whether kernels launched from now on may begin (their prologue, up to `pdl_wait`) before the kernel before them has ended
+    (csrc/common.cuh, programmatic dependent launch).  A launch recorded in a graph keeps what held when it was recorded."""
+    global _overlap
+    on = bool(on)
+    if on == _overlap:
+        return
+    with _lock:
+        _overlap = on
+        for lib in _loaded.values():
+            _set_overlap_of(lib)
 
 
 def build_all(verbose: bool = True, jobs: int = 4) -> Dict[str, str]:

@@ -63,7 +63,15 @@ static inline int launch_status() { return (int)cudaGetLastError(); }
 __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 
+//
+// `llmx_launch_overlap` (one per library, exported; build.py `set_overlap` writes it): 0 launches without the attribute, so
+// that a kernel starts when everything before it on the stream has ended.
+extern "C" {
+__attribute__((visibility("default"), weak)) int llmx_launch_overlap = 1;
+}
+
 static inline bool llmx_pdl_enabled() {
+    if (!llmx_launch_overlap) return false;
     static int on = -1;
     if (on < 0) {
         const char* e = getenv("LLMX_PDL");

@@ -27,10 +27,17 @@ import numpy as np
 import torch
 
 from .. import runtime
+from ..csrc import build as _build
 from ..parts.base import NativeHandle, Part, PartPlan, Precision, StepBatch, StepShape, tensor_name
 from ..parts.embedding import LogitsHead, TokenEmbedding
 from ..weights.loader import check_tensors, stored
 from ..weights.spec import TensorSpec
+
+
+# A step of more rows than this, walked from Python, launches its kernels one strictly after the other.  (With few rows the
+# products are short and the overlap of their prologues shows; with many, and the host launching each kernel by itself,
+# it gains next to nothing, and prompt steps of such models have been seen to stall with it.)
+OVERLAP_MAX_ROWS = 64
 
 
 @dataclass(frozen=True)
@@ -261,6 +268,13 @@ class Model:
     def forward(self, step: StepBatch) -> Optional[torch.Tensor]:
         """Run the step's rows through every layer; logits [wanted, vocab] float32, or None if none is wanted."""
         wanted = step.logit_rows.numel()
+        _build.set_overlap(self.native is not None or step.rows <= OVERLAP_MAX_ROWS)
+        try:
+            return self._forward(step, wanted)
+        finally:
+            _build.set_overlap(True)
+
+    def _forward(self, step: StepBatch, wanted: int) -> Optional[torch.Tensor]:
         if self.native is not None:
             rt = runtime.lib()
             probe = step.struct_for(self)

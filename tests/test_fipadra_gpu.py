@@ -652,3 +652,19 @@ def test_trace_run_program(tmp_path):
         refs, skip = references(cfg, w, requests, 0.03 if dtype == "bfloat16" else None)
         worst, where = worst_error(got, refs, skip)
         assert worst <= tol * max(float(np.abs(r).max()) for r in refs.values()), (dtype, worst, where)
+
+
+def test_steps_of_many_rows_launch_strictly_in_order(tmp_path):
+    """A model walked from Python lets kernels begin before the ones before them have ended in steps of few rows only."""
+    from llmx_b200.csrc import build
+    from llmx_b200.engine import StepEntry
+    from llmx_b200.models.model import OVERLAP_MAX_ROWS
+    cfg = config([ret(heads=2, dim=8, vdim=8)])
+    make_folder(str(tmp_path), cfg, seed=1)
+    e = engine_of(str(tmp_path), "float32", 256)
+    seen, forward = [], e.model.blocks[0].forward
+    e.model.blocks[0].forward = lambda *a, **k: (seen.append(build._overlap), forward(*a, **k))
+    for n in (1, OVERLAP_MAX_ROWS, OVERLAP_MAX_ROWS + 1):
+        e.step([StepEntry("r", helpers.random_ids(cfg["vocab"], n, seed=n), [0])])
+        e.end("r")
+    assert seen == [True, True, False] and build._overlap
