@@ -6,5 +6,6 @@ from .kisepel import KisepelConfig
 from .zamizen import ZamizenConfig
 from .nomutar import NomutarConfig
 from .fipadra import FipadraConfig
+from .dikusun import DikusunConfig
 
-__all__ = ["ConfigError", "ModelConfig", "Rule", "apply_rules", "read_config_json", "Qwen3Config", "YarnScaling", "BuzetarConfig", "KisepelConfig", "ZamizenConfig", "NomutarConfig", "FipadraConfig"]
+__all__ = ["ConfigError", "ModelConfig", "Rule", "apply_rules", "read_config_json", "Qwen3Config", "YarnScaling", "BuzetarConfig", "KisepelConfig", "ZamizenConfig", "NomutarConfig", "FipadraConfig", "DikusunConfig"]

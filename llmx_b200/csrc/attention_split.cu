@@ -5,7 +5,10 @@
 // weight of D values shared by the heads (optional), a rotation of the first 2 * rot_half values of every query and
 // key head (value i pairs with value i + rot_half; the angle is position * freq[i], made in 32-bit here, so there is
 // no table whose length bounds the context), queries to `q_out`, keys and values to the row's cache slot.
-// Designs vary the softmax (`AttnExtras`: a cap on the scores, a sink in the denominator, values rotated by position).
+// Designs vary the softmax (`AttnExtras`: a cap on the scores, a sink in the denominator, values rotated by position, a gate
+// per head on the output, and differential attention: two maps per head over the same values, of which the second is
+// subtracted from the first).  With two maps a cache row is [key of map 1 ; key of map 2 ; value], queries and keys lie head
+// by head as [map 1, map 2], and every kernel here serves "map heads": map head 2 h + n is map n of head h.
 // `llmx_attention_split` is the plain form of the attention: one block per (row, head); a row at position p reads the
 // keys lo..p of its own request, where lo is the larger of p - window + 1 (window > 0) and the start of p's chunk,
 // floor(p / chunk) * chunk (chunk > 0: positions are counted from the start of the request, so chunks do not move
@@ -114,6 +117,7 @@ struct QkvFinish {
     const int *positions, *slots;
     int heads, kv_heads, D, V, page_size, rows;
     int planes;   // 1: a slot holds [key ; value] in one row of D + V; 2: keys and values in planes of their own (D = V)
+    int maps;             // keys a key/value head has in a cache row (`heads` counts queries per map: heads * maps of them)
     float rot_mag;        // a factor on the cosines and sines of the q/k rotation
     const float* vfreq;   // [V / 2] or null: values are rotated by their position over all of V, in the q/k pairing
 };
@@ -127,7 +131,8 @@ qkv_finish_kernel(QkvFinish a, QT* __restrict__ q_out, KVT* __restrict__ cache) 
     __shared__ float turn[2][16 * MAX_PER_LANE];
     const int keep = a.taps - 1;
     const int D = a.D, V = a.V;
-    const int channels = (a.heads + a.kv_heads) * D + a.kv_heads * V;
+    const int k_heads = a.kv_heads * a.maps;
+    const int channels = (a.heads + k_heads) * D + a.kv_heads * V;
     if ((int)blockIdx.x >= a.rows) {
         // The filter's inputs a later step needs: the last `keep` values of u of the request, from this step's rows or,
         // when the step brings fewer, from the slot read (the slot written is another one).
@@ -178,7 +183,7 @@ qkv_finish_kernel(QkvFinish a, QT* __restrict__ q_out, KVT* __restrict__ cache) 
     __shared__ float whole[2], whole_part[4];
     if (a.norm == 3) {
         for (int which = 0; which < (a.kv_heads > 0 ? 2 : 1); ++which) {
-            const int c_lo = which == 0 ? 0 : a.heads * D, c_hi = which == 0 ? a.heads * D : (a.heads + a.kv_heads) * D;
+            const int c_lo = which == 0 ? 0 : a.heads * D, c_hi = which == 0 ? a.heads * D : (a.heads + k_heads) * D;
             float ss = 0.0f;
             for (int c = c_lo + threadIdx.x; c < c_hi; c += blockDim.x) {
                 const float v = filtered(c);
@@ -197,8 +202,8 @@ qkv_finish_kernel(QkvFinish a, QT* __restrict__ q_out, KVT* __restrict__ cache) 
     }
     __syncthreads();
     float* st = stage[warp];
-    const int v_off = (a.heads + a.kv_heads) * D;
-    for (int item = blockIdx.y * warps + warp; item < a.heads + a.kv_heads; item += gridDim.y * warps) {
+    const int v_off = (a.heads + k_heads) * D;
+    for (int item = blockIdx.y * warps + warp; item < a.heads + k_heads; item += gridDim.y * warps) {
         const bool is_q = item < a.heads;
         if (!is_q && slot < 0) continue;                              // a row whose cache write is skipped
         const float* w = is_q ? a.q_weight : a.k_weight;
@@ -234,13 +239,16 @@ qkv_finish_kernel(QkvFinish a, QT* __restrict__ q_out, KVT* __restrict__ cache) 
             QT* dst = q_out + ((size_t)row * a.heads + item) * D;
             for (int d = lane; d < D; d += 32) dst[d] = from_float<QT>(a.norm == 2 ? st[d] * rr * (w ? w[d] : 1.0f) : st[d]);
         } else {
-            const int g = item - a.heads;
+            const int g = (item - a.heads) / a.maps, map = (item - a.heads) % a.maps;
             const size_t page = slot / a.page_size, off = slot % a.page_size;
             KVT* dst = a.planes == 2 ? cache + (((page * 2) * a.kv_heads + g) * a.page_size + off) * (size_t)D
-                                     : cache + ((page * a.kv_heads + g) * a.page_size + off) * (size_t)(D + V);
-            KVT* vdst = a.planes == 2 ? dst + (size_t)a.kv_heads * a.page_size * D : dst + D;
+                                     : cache + ((page * a.kv_heads + g) * a.page_size + off) * (size_t)(a.maps * D + V);
+            KVT* vdst = a.planes == 2 ? dst + (size_t)a.kv_heads * a.page_size * D : dst + a.maps * D;
+            dst += map * D;
             for (int d = lane; d < D; d += 32) dst[d] = from_float<KVT>(a.norm == 2 ? st[d] * rr * (w ? w[d] : 1.0f) : st[d]);
-            if (a.vfreq == nullptr) {
+            if (map > 0) {
+                // the head's first map writes its value
+            } else if (a.vfreq == nullptr) {
                 for (int d = lane; d < V; d += 32) vdst[d] = from_float<KVT>(filtered(v_off + g * V + d));
             } else {
                 __syncwarp();                                         // the key has left the stage
@@ -266,13 +274,31 @@ qkv_finish_kernel(QkvFinish a, QT* __restrict__ q_out, KVT* __restrict__ cache) 
 //             2: the same with 0 for every head (one is added to the denominator)
 //   vfreq [V / 2]: the cached values were rotated by their positions over all of V (pair m by position * vfreq[m]; pairs
 //             (m, m + V / 2), or with v_neighbours (2m, 2m + 1)); a row's output is turned back by its own position
+//   gate [rows, gate_stride]: head h's output times sigmoid(gate[row, h])
+//   maps 2: with a1, a2 the attentions of a head's two maps, o = a1 - factor * a2, then o / sqrt(mean(o^2) + eps) over the V
+//             values, times out_factor (and the gate); no sink and no rotated values then
 struct AttnExtras {
     float softcap;
     const float* sink;
     int sink_mode;
     const float* vfreq;
     int v_neighbours;
+    int maps;
+    float factor, out_factor, eps;
+    const float* gate;
+    int gate_stride;
 };
+
+static bool extras_fit(const AttnExtras& x, int heads, int kv_heads, int V) {
+    if (x.sink_mode < 0 || x.sink_mode > 2 || (x.sink_mode == 1 && x.sink == nullptr) || (x.vfreq != nullptr && V % 2)) return false;
+    if (x.maps != 1 && (x.maps != 2 || x.sink_mode || x.vfreq != nullptr)) return false;
+    if (x.gate != nullptr && x.gate_stride < heads / x.maps) return false;
+    return kv_heads > 0 && heads > 0 && heads % kv_heads == 0 && (heads / kv_heads) % x.maps == 0;
+}
+
+__device__ __forceinline__ float head_gate(const AttnExtras& x, int row, int head) {
+    return x.gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-x.gate[(size_t)row * x.gate_stride + head]));
+}
 
 // The factor on the weighted sum and the whole denominator, given the keys' maximum m and sum l (relative to m).
 __device__ __forceinline__ float finish_softmax(float m, float l, const AttnExtras& x, int head) {
@@ -313,7 +339,8 @@ attention_split_kernel(const QT* __restrict__ q, const KVT* __restrict__ cache, 
     int lo = window > 0 ? max(0, pos - window + 1) : 0;
     if (chunk > 0) lo = max(lo, (pos / chunk) * chunk);
     const int* table = block_tables + (size_t)row_request[row] * table_stride;
-    const int W = D + V;
+    const int W = extras.maps * D + V, k_off = (h % extras.maps) * D, v_off = extras.maps * D;
+    const bool leave_partial = splits > 1 || extras.maps > 1;
 
     float qv[MAX_PER_LANE], acc[MAX_PER_LANE];
     const QT* qrow = q + ((size_t)row * heads + h) * D;
@@ -334,8 +361,8 @@ attention_split_kernel(const QT* __restrict__ q, const KVT* __restrict__ cache, 
     }
     for (int t = first + warp; t <= last; t += WARPS) {
         const int page = table[t / page_size], off = t % page_size;
-        const KVT* kp = cache + (((size_t)page * kv_heads + g) * page_size + off) * (size_t)W;
-        const KVT* vp = kp + D;
+        const KVT* kp = cache + (((size_t)page * kv_heads + g) * page_size + off) * (size_t)W + k_off;
+        const KVT* vp = kp - k_off + v_off;
         float s = 0.0f;
 #pragma unroll
         for (int i = 0; i < MAX_PER_LANE; ++i) {
@@ -376,7 +403,7 @@ attention_split_kernel(const QT* __restrict__ q, const KVT* __restrict__ cache, 
             f[w] = mw == -INFINITY ? 0.0f : expf(mw - mm);
             ll += smem[w * (V + 2) + V + 1] * f[w];
         }
-        if (splits > 1) {
+        if (leave_partial) {
             float* prow = partial + (((size_t)row * heads + h) * splits + blockIdx.z) * (size_t)(V + 2);
             for (int d = lane; d < V; d += 32) {
                 float o = 0.0f;
@@ -390,7 +417,7 @@ attention_split_kernel(const QT* __restrict__ q, const KVT* __restrict__ cache, 
             return;
         }
         QT* orow = out + ((size_t)row * heads + h) * V;
-        const float inv = finish_softmax(mm, ll, extras, h);
+        const float inv = finish_softmax(mm, ll, extras, h) * head_gate(extras, row, h);
         float* turned = smem + WARPS * (V + 2);
         for (int d = lane; d < V; d += 32) {
             float o = 0.0f;
@@ -424,7 +451,7 @@ attention_merge_kernel(const float* __restrict__ partial, QT* __restrict__ out, 
         const float ms = p[(size_t)s * (V + 2) + V];
         ll += ms == -INFINITY ? 0.0f : p[(size_t)s * (V + 2) + V + 1] * expf(ms - mm);
     }
-    const float inv = finish_softmax(mm, ll, extras, item % heads);
+    const float inv = finish_softmax(mm, ll, extras, item % heads) * head_gate(extras, item / heads, item % heads);
     for (int d = lane; d < V; d += 32) {
         float o = 0.0f;
         for (int s = 0; s < splits; ++s) {
@@ -438,6 +465,68 @@ attention_merge_kernel(const float* __restrict__ partial, QT* __restrict__ out, 
         __syncwarp();
         write_turned_back(turned, out + (size_t)item * V, V, (float)positions[item / heads], extras, lane);
     }
+}
+
+// The two maps of one (row, head) merged and combined (see `AttnExtras`).  One warp a (row, head); `heads` counts heads.
+template <typename QT>
+__global__ void __launch_bounds__(128)
+attention_merge_maps_kernel(const float* __restrict__ partial, QT* __restrict__ out, int items, int V, int splits, int heads,
+                            AttnExtras extras) {
+    pdl_trigger();
+    pdl_wait();
+    const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= items) return;
+    float o[MAX_PER_LANE];
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) o[i] = 0.0f;
+    for (int map = 0; map < 2; ++map) {
+        const float* p = partial + ((size_t)item * 2 + map) * splits * (V + 2);
+        float mm = -INFINITY;
+        for (int s = 0; s < splits; ++s) mm = fmaxf(mm, p[(size_t)s * (V + 2) + V]);
+        float ll = 0.0f;
+        for (int s = 0; s < splits; ++s) {
+            const float ms = p[(size_t)s * (V + 2) + V];
+            ll += ms == -INFINITY ? 0.0f : p[(size_t)s * (V + 2) + V + 1] * expf(ms - mm);
+        }
+        const float inv = (map == 0 ? 1.0f : -extras.factor) / ll;
+        for (int s = 0; s < splits; ++s) {
+            const float ms = p[(size_t)s * (V + 2) + V];
+            if (ms == -INFINITY) continue;
+            const float f = expf(ms - mm) * inv;
+#pragma unroll
+            for (int i = 0; i < MAX_PER_LANE; ++i) {
+                const int d = lane + 32 * i;
+                if (d < V) o[i] = fmaf(p[(size_t)s * (V + 2) + d], f, o[i]);
+            }
+        }
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) ss = fmaf(o[i], o[i], ss);
+    const float f = extras.out_factor / sqrtf(warp_sum(ss) / (float)V + extras.eps) * head_gate(extras, item / heads, item % heads);
+    QT* orow = out + (size_t)item * V;
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) {
+        const int d = lane + 32 * i;
+        if (d < V) orow[d] = from_float<QT>(o[i] * f);
+    }
+}
+
+// The merge of `heads` map heads' ranges, whichever form left them.
+static int launch_merge(const float* partial, void* out, int q_dtype, int rows, int heads, int V, int splits, const int* positions,
+                        const AttnExtras& extras, cudaStream_t stream) {
+    const int items = rows * heads / extras.maps;
+    const dim3 grid((items + 3) / 4);
+    const size_t smem = (size_t)4 * V * sizeof(float);
+    if (extras.maps == 2) {
+        if (q_dtype == LLMX_BF16) launch_kernel(attention_merge_maps_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, partial, (__nv_bfloat16*)out, items, V, splits, heads / 2, extras);
+        else launch_kernel(attention_merge_maps_kernel<float>, grid, dim3(128), 0, stream, partial, (float*)out, items, V, splits, heads / 2, extras);
+    } else if (q_dtype == LLMX_BF16) {
+        launch_kernel(attention_merge_kernel<__nv_bfloat16>, grid, dim3(128), smem, stream, partial, (__nv_bfloat16*)out, items, V, splits, heads, positions, extras);
+    } else {
+        launch_kernel(attention_merge_kernel<float>, grid, dim3(128), smem, stream, partial, (float*)out, items, V, splits, heads, positions, extras);
+    }
+    return launch_status();
 }
 
 // ---- the staged form, for rows that are few -------------------------------------------------------------------------------
@@ -474,13 +563,13 @@ __global__ void __launch_bounds__(128)
 attention_staged_kernel(const T* __restrict__ q, const T* __restrict__ cache, const int* __restrict__ row_request,
                         const int* __restrict__ positions, const int* __restrict__ block_tables, int table_stride, int heads,
                         int kv_heads, int D, int V, int page_size, int window, int chunk, float scale, int splits, int TK,
-                        float softcap, float* __restrict__ partial) {
+                        float softcap, int maps, float* __restrict__ partial) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char st_smem[];
     constexpr int EP = Piece<T>::N;
     const int row = blockIdx.x, g = blockIdx.y, split = blockIdx.z;
-    const int ratio = heads / kv_heads, W = D + V, ws = W + EP, pieces = W / EP;
+    const int ratio = heads / kv_heads, W = maps * D + V, ws = W + EP, pieces = W / EP;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* qs = reinterpret_cast<float*>(st_smem);               // [ratio][D]
     float* ps = qs + (size_t)ratio * D;                          // [ratio][TK]
@@ -532,7 +621,7 @@ attention_staged_kernel(const T* __restrict__ q, const T* __restrict__ cache, co
             float* ph = ps + (size_t)hl * TK;
             float mx = -INFINITY;
             for (int kt = lane; kt < TK; kt += 32) {
-                const T* kr = buf + (size_t)kt * ws;
+                const T* kr = buf + (size_t)kt * ws + (hl % maps) * D;
                 float s = 0.0f;
                 for (int d = 0; d < D; d += EP) {
                     float kvv[EP];
@@ -568,7 +657,7 @@ attention_staged_kernel(const T* __restrict__ q, const T* __restrict__ cache, co
             __syncwarp();
             for (int key = 0; key < n_here; ++key) {
                 const float e = ph[key];
-                const T* vr = buf + (size_t)key * ws + D;
+                const T* vr = buf + (size_t)key * ws + maps * D;
 #pragma unroll
                 for (int i = 0; i < VPL; ++i) {
                     const int c = lane + 32 * i;
@@ -598,14 +687,14 @@ attention_staged_kernel(const T* __restrict__ q, const T* __restrict__ cache, co
 
 // The tile of keys the staged form takes for these sizes (the largest of 64, 32, 16 whose buffers fit), or 0 when it does
 // not take them: equal types of queries and cache, key and whole-row widths in 16-byte pieces, at most 16 heads a group.
-static int staged_tile(int q_dtype, int cache_dtype, int heads, int kv_heads, int D, int V, size_t* smem_out) {
+static int staged_tile(int q_dtype, int cache_dtype, int heads, int kv_heads, int D, int V, int maps, size_t* smem_out) {
     if (q_dtype != cache_dtype || (q_dtype != LLMX_BF16 && q_dtype != LLMX_F32)) return 0;
     if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || heads / kv_heads > 16 || D <= 0 || V <= 0 || V > 512 || D > 512) return 0;
     const int ep = q_dtype == LLMX_BF16 ? 8 : 4, es = q_dtype == LLMX_BF16 ? 2 : 4;
-    if (D % ep || (D + V) % ep) return 0;
+    if (D % ep || V % ep || maps < 1 || maps > 2) return 0;
     const int ratio = heads / kv_heads;
     for (int tk = 64; tk >= 16; tk /= 2) {
-        const size_t smem = ((size_t)ratio * D + (size_t)ratio * tk) * 4 + 2 * (size_t)tk * (D + V + ep) * es;
+        const size_t smem = ((size_t)ratio * D + (size_t)ratio * tk) * 4 + 2 * (size_t)tk * (maps * D + V + ep) * es;
         if (smem <= 72 * 1024) {
             if (smem_out) *smem_out = smem;
             return tk;
@@ -649,8 +738,8 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t& a, uint32_t& 
     c = *reinterpret_cast<uint32_t*>(&p2);
 }
 
-template <int VN_MAX>
-__global__ void __launch_bounds__(128)
+template <int VN_MAX, int MAPS>
+__global__ void __launch_bounds__(128, VN_MAX <= 8 ? 3 : 1)
 attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache,
                        __nv_bfloat16* __restrict__ out, const int* __restrict__ row_start, const int* __restrict__ row_count,
                        const int* __restrict__ history, const int* __restrict__ block_tables, int table_stride, int requests,
@@ -659,7 +748,8 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char tl_smem[];
-    const int ratio = heads / kv_heads, tok = TL_ROWS / r_pad;
+    constexpr int MAP_ROWS = TL_ROWS / MAPS;
+    const int ratio = heads / kv_heads / MAPS, tok = MAP_ROWS / r_pad;
     // Which tile: the requests' tiles are numbered one request after the other.
     int idx = blockIdx.x, r = 0, tiles_r = 0;
     for (; r < requests; ++r) {
@@ -672,7 +762,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
     const int g = blockIdx.y;
     const int t0 = idx * tok, n_rows = row_count[r], a0 = row_start[r], hist = history[r];
     const int n_tok = min(tok, n_rows - t0);
-    const int W = D + V, qs = D + TL_PAD, ws = W + TL_PAD;
+    const int W = MAPS * D + V, qs = D + TL_PAD, ws = W + TL_PAD;
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(tl_smem);
     __nv_bfloat16* KV = Qs + (size_t)TL_ROWS * qs;               // [2][TL_KEYS][ws]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
@@ -704,14 +794,15 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     issue(0, 0);
-    // The tile's queries: row i is token t0 + i / r_pad, head g * ratio + i % r_pad (rows past the heads or the tokens are zeros).
+    // The tile's queries: row i is token t0 + i / r_pad, head g * ratio + i % r_pad (rows past the heads or the tokens are zeros);
+    // with two maps the rows' first half is the first map's and the second half the second's.
     const int d8 = D / 8;
     for (int i = threadIdx.x; i < TL_ROWS * d8; i += 128) {
         const int row = i / d8, c = i - row * d8;
-        const int tk = row / r_pad, hd = row % r_pad;
+        const int tk = row % MAP_ROWS / r_pad, hd = row % r_pad, map = row / MAP_ROWS;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (tk < n_tok && hd < ratio)
-            v = *reinterpret_cast<const uint4*>(q + ((size_t)(a0 + t0 + tk) * heads + (size_t)g * ratio + hd) * D + 8 * c);
+            v = *reinterpret_cast<const uint4*>(q + ((size_t)(a0 + t0 + tk) * heads + ((size_t)g * ratio + hd) * MAPS + map) * D + 8 * c);
         *reinterpret_cast<uint4*>(Qs + (size_t)row * qs + 8 * c) = v;
     }
     bool valid[2];
@@ -719,7 +810,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
     for (int hf = 0; hf < 2; ++hf) {
         const int row = 16 * warp + gid + 8 * hf;
-        const int tk = row / r_pad, hd = row % r_pad;
+        const int tk = row % MAP_ROWS / r_pad, hd = row % r_pad;
         valid[hf] = tk < n_tok && hd < ratio;
         pos[hf] = hist + t0 + tk;
         lo[hf] = lowest(pos[hf]);
@@ -729,6 +820,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
     for (int i = 0; i < VN_MAX; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     const int vn = V / 8;
+    const int k_off = MAPS == 1 ? 0 : (16 * warp / MAP_ROWS) * D;    // a warp's rows are all of one map
     for (int tile = 0; tile < n_tiles; ++tile) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                 // this tile has landed (and the queries); everyone has left the other buffer
@@ -747,7 +839,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             a[3] = *reinterpret_cast<const uint32_t*>(qa + 8 * qs + 8);
 #pragma unroll
             for (int n = 0; n < 8; ++n) {
-                const __nv_bfloat16* kb = buf + (size_t)(8 * n + gid) * ws + kk + 2 * tig;
+                const __nv_bfloat16* kb = buf + (size_t)(8 * n + gid) * ws + k_off + kk + 2 * tig;
                 mma_bf16_16816(s[n], a, *reinterpret_cast<const uint32_t*>(kb), *reinterpret_cast<const uint32_t*>(kb + 8));
             }
         }
@@ -795,7 +887,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             split3(s[2 * ks][2], s[2 * ks][3], p0[1], p1[1], p2[1]);
             split3(s[2 * ks + 1][0], s[2 * ks + 1][1], p0[2], p1[2], p2[2]);
             split3(s[2 * ks + 1][2], s[2 * ks + 1][3], p0[3], p1[3], p2[3]);
-            const __nv_bfloat16* vrow = buf + (size_t)(16 * ks + (lane & 15)) * ws + D;
+            const __nv_bfloat16* vrow = buf + (size_t)(16 * ks + (lane & 15)) * ws + MAPS * D;
 #pragma unroll
             for (int nv = 0; nv < VN_MAX; ++nv) {
                 if (nv < vn) {
@@ -809,6 +901,53 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             }
         }
     }
+    if constexpr (MAPS == 2) {
+        // The second map's warps leave their attention in shared memory (the key buffers are free now); the first map's take
+        // the difference, norm it over the head's values and store it.
+        float* second = reinterpret_cast<float*>(KV);                // [MAP_ROWS][V + 2]
+        const int vs = V + 2;
+        __syncthreads();
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+            l[hf] += __shfl_xor_sync(0xffffffffu, l[hf], 1);
+            l[hf] += __shfl_xor_sync(0xffffffffu, l[hf], 2);
+            const float inv = valid[hf] ? 1.0f / l[hf] : 0.0f;
+            const int row = (16 * warp + gid + 8 * hf) % MAP_ROWS;
+#pragma unroll
+            for (int nv = 0; nv < VN_MAX; ++nv) {
+                if (nv >= vn) continue;
+                o[nv][2 * hf] *= inv;
+                o[nv][2 * hf + 1] *= inv;
+                if (16 * warp >= MAP_ROWS) *reinterpret_cast<float2*>(second + row * vs + 8 * nv + 2 * tig) = make_float2(o[nv][2 * hf], o[nv][2 * hf + 1]);
+            }
+        }
+        __syncthreads();
+        if (16 * warp >= MAP_ROWS) return;
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+            const int row = 16 * warp + gid + 8 * hf, tk = row / r_pad, hd = row % r_pad;
+            float ss = 0.0f;
+#pragma unroll
+            for (int nv = 0; nv < VN_MAX; ++nv) {
+                if (nv >= vn) continue;
+                const float2 b = *reinterpret_cast<const float2*>(second + row * vs + 8 * nv + 2 * tig);
+                o[nv][2 * hf] = fmaf(-extras.factor, b.x, o[nv][2 * hf]);
+                o[nv][2 * hf + 1] = fmaf(-extras.factor, b.y, o[nv][2 * hf + 1]);
+                ss = fmaf(o[nv][2 * hf], o[nv][2 * hf], ss);
+                ss = fmaf(o[nv][2 * hf + 1], o[nv][2 * hf + 1], ss);
+            }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            if (!valid[hf]) continue;
+            const float f = extras.out_factor / sqrtf(ss / (float)V + extras.eps) * head_gate(extras, a0 + t0 + tk, g * ratio + hd);
+            __nv_bfloat16* orow = out + ((size_t)(a0 + t0 + tk) * (heads / 2) + (size_t)g * ratio + hd) * V;
+#pragma unroll
+            for (int nv = 0; nv < VN_MAX; ++nv)
+                if (nv < vn)
+                    *reinterpret_cast<uint32_t*>(orow + 8 * nv + 2 * tig) = pack_bf16(o[nv][2 * hf] * f, o[nv][2 * hf + 1] * f);
+        }
+        return;
+    }
     if (extras.vfreq) {
         // Rotated values: the normed outputs meet in shared memory (the key buffers are free now), and every row is turned
         // back by its own position on the way out.
@@ -819,7 +958,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
             l[hf] += __shfl_xor_sync(0xffffffffu, l[hf], 1);
             l[hf] += __shfl_xor_sync(0xffffffffu, l[hf], 2);
             const int row = 16 * warp + gid + 8 * hf;
-            const float inv = valid[hf] ? finish_softmax(m[hf], l[hf], extras, g * ratio + row % r_pad) : 0.0f;
+            const float inv = valid[hf] ? finish_softmax(m[hf], l[hf], extras, g * ratio + row % r_pad) * head_gate(extras, a0 + t0 + row / r_pad, g * ratio + row % r_pad) : 0.0f;
 #pragma unroll
             for (int nv = 0; nv < VN_MAX; ++nv)
                 if (nv < vn) {
@@ -850,7 +989,7 @@ attention_tiled_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
         if (!valid[hf]) continue;
         const int row = 16 * warp + gid + 8 * hf;
         const int tk = row / r_pad, hd = row % r_pad;
-        const float inv = finish_softmax(m[hf], l[hf], extras, g * ratio + hd);
+        const float inv = finish_softmax(m[hf], l[hf], extras, g * ratio + hd) * head_gate(extras, a0 + t0 + tk, g * ratio + hd);
         __nv_bfloat16* orow = out + ((size_t)(a0 + t0 + tk) * heads + (size_t)g * ratio + hd) * V;
 #pragma unroll
         for (int nv = 0; nv < VN_MAX; ++nv)
@@ -892,26 +1031,28 @@ LLMX_EXPORT int llmx_qk_norm_rope_write(const float* proj, int stride, const flo
 // [rot_pairs], cosines and sines times rot_mag; vfreq float32 [V / 2] or null: values rotated over all of V by their position;
 // the rows' requests, their row ranges, histories and the slots read and written as a step gives them.
 // planes 1: cache [pages, 1, kv_heads, page_size, D + V]; planes 2 (D = V): cache [pages, 2, kv_heads, page_size, D], the
-// layout of the paged kernels with key and value planes.
+// layout of the paged kernels with key and value planes.  maps n: `heads` query heads and kv_heads * maps key heads, the latter
+// in cache rows of n keys and one value, [pages, 1, kv_heads, page_size, n D + V].
 LLMX_EXPORT int llmx_qkv_finish(const float* proj, int stride, const float* bias, const float* taps_w, int taps, float* state,
                                 long long slot_floats, long long conv_off, const int* row_request, const int* row_start,
                                 const int* row_count, const int* history, const int* slot_in, const int* slot_out,
                                 const float* q_weight, const float* k_weight, int norm, float eps, const float* freq, int rot_pairs,
                                 int neighbours, const int* positions, const int* slots, void* q_out, int q_dtype, void* cache,
                                 int cache_dtype, int rows, int requests, int heads, int kv_heads, int D, int V, int page_size,
-                                int planes, float rot_mag, const float* vfreq, cudaStream_t stream) {
+                                int planes, int maps, float rot_mag, const float* vfreq, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (planes != 1 && !(planes == 2 && D == V)) return LLMX_ERR_BAD_ARGUMENT;
+    if (maps < 1 || (maps > 1 && planes != 1)) return LLMX_ERR_BAD_ARGUMENT;
     if (D <= 0 || V <= 0 || heads <= 0 || kv_heads < 0 || D > 32 * MAX_PER_LANE || 2 * rot_pairs > D || rot_pairs < 0 ||
         (rot_pairs > 0 && freq == nullptr) || norm < 0 || norm > 3 || taps < 1 || (vfreq != nullptr && (V % 2 || V > 32 * MAX_PER_LANE)) || (taps > 1 && (taps_w == nullptr || state == nullptr)) ||
         (kv_heads > 0 && (cache == nullptr || slots == nullptr || page_size <= 0)))
         return LLMX_ERR_BAD_ARGUMENT;
-    const long long channels = (long long)(heads + kv_heads) * D + (long long)kv_heads * V;
+    const long long channels = ((long long)heads + (long long)kv_heads * maps) * D + (long long)kv_heads * V;
     if (taps > 1 && conv_off + (taps - 1) * channels > slot_floats) return LLMX_ERR_BAD_ARGUMENT;
     QkvFinish a{proj, stride, bias, taps_w, taps, state, slot_floats, conv_off, row_request, row_start, row_count, history, slot_in,
                 slot_out, q_weight, k_weight, norm, eps, freq, rot_pairs, neighbours, positions, slots, heads, kv_heads, D, V,
-                page_size > 0 ? page_size : 1, rows, planes, rot_mag, vfreq};
-    const dim3 grid(rows + (taps > 1 ? requests : 0), std::min((heads + kv_heads + 3) / 4, 64));
+                page_size > 0 ? page_size : 1, rows, planes, maps, rot_mag, vfreq};
+    const dim3 grid(rows + (taps > 1 ? requests : 0), std::min((heads + kv_heads * maps + 3) / 4, 64));
     const bool cache16 = kv_heads > 0 && cache_dtype == LLMX_BF16;
     if (kv_heads > 0 && cache_dtype != LLMX_BF16 && cache_dtype != LLMX_F32) return LLMX_ERR_UNSUPPORTED;
     if (q_dtype == LLMX_BF16 && cache16) launch_kernel(qkv_finish_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(128), 0, stream, a, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache);
@@ -922,20 +1063,21 @@ LLMX_EXPORT int llmx_qkv_finish(const float* proj, int stride, const float* bias
     return launch_status();
 }
 
-// q [rows, heads, D] and out [rows, heads, V] of `q_dtype`; the cache as above, of `cache_dtype`.  `splits` > 1: a row's
+// q [rows, heads, D] and out [rows, heads / maps, V] of `q_dtype`; the cache as above, of `cache_dtype`.  `splits` > 1: a row's
 // keys are cut into that many ranges (a matter of speed only: steps of few rows over long histories), which meet in
-// `partial`, float32 [rows, heads, splits, V + 2].
+// `partial`, float32 [rows, heads, splits, V + 2] (with two maps in any case).  `maps` 2: `heads` counts map heads.
 LLMX_EXPORT int llmx_attention_split(const void* q, int q_dtype, const void* cache, int cache_dtype, void* out,
                                      const int* row_request, const int* positions, const int* block_tables,
                                      int table_stride, int rows, int heads, int kv_heads, int D, int V, int page_size,
                                      int window, int chunk, float scale, int splits, float* partial, float softcap,
-                                     const float* sink, int sink_mode, const float* vfreq, int v_neighbours, cudaStream_t stream) {
+                                     const float* sink, int sink_mode, const float* vfreq, int v_neighbours, int maps, float factor,
+                                     float out_factor, float eps, const float* gate, int gate_stride, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (sink_mode < 0 || sink_mode > 2 || (sink_mode == 1 && sink == nullptr) || (vfreq != nullptr && V % 2)) return LLMX_ERR_BAD_ARGUMENT;
-    const AttnExtras extras{softcap, sink, sink_mode, vfreq, v_neighbours};
+    const AttnExtras extras{softcap, sink, sink_mode, vfreq, v_neighbours, maps, factor, out_factor, eps, gate, gate_stride};
+    if (!extras_fit(extras, heads, kv_heads, V)) return LLMX_ERR_BAD_ARGUMENT;
     if (D <= 0 || V <= 0 || D > 32 * MAX_PER_LANE || V > 32 * MAX_PER_LANE || heads % kv_heads || heads > 65535)
         return LLMX_ERR_UNSUPPORTED;
-    if (splits < 1 || splits > 64 || (splits > 1 && partial == nullptr)) return LLMX_ERR_BAD_ARGUMENT;
+    if (splits < 1 || splits > 64 || ((splits > 1 || maps > 1) && partial == nullptr)) return LLMX_ERR_BAD_ARGUMENT;
     dim3 grid(rows, heads, splits);
     const size_t shmem = ((size_t)WARPS * (V + 2) + V) * sizeof(float);
 #define LLMX_SPLIT(QT, KVT)                                                                                            \
@@ -949,21 +1091,19 @@ LLMX_EXPORT int llmx_attention_split(const void* q, int q_dtype, const void* cac
     else return LLMX_ERR_UNSUPPORTED;
 #undef LLMX_SPLIT
     int status = launch_status();
-    if (status || splits == 1) return status;
-    const int items = rows * heads;
-    if (q_dtype == LLMX_BF16)
-        launch_kernel(attention_merge_kernel<__nv_bfloat16>, dim3((items + 3) / 4), dim3(128), (size_t)4 * V * sizeof(float), stream, (const float*)partial, (__nv_bfloat16*)out, items, V, splits, heads, positions, extras);
-    else
-        launch_kernel(attention_merge_kernel<float>, dim3((items + 3) / 4), dim3(128), (size_t)4 * V * sizeof(float), stream, (const float*)partial, (float*)out, items, V, splits, heads, positions, extras);
-    return launch_status();
+    if (status || (splits == 1 && maps == 1)) return status;
+    return launch_merge(partial, out, q_dtype, rows, heads, V, splits, positions, extras, stream);
 }
 
 // Whether the tiled form takes these sizes (bfloat16 queries and cache are the caller's to check).
-LLMX_EXPORT int llmx_attention_tiled_fits(int heads, int kv_heads, int D, int V) {
-    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || heads / kv_heads > TL_ROWS) return 0;
+static size_t tiled_smem(int D, int V, int maps) {
+    return ((size_t)TL_ROWS * (D + TL_PAD) + 2 * (size_t)TL_KEYS * (maps * D + V + TL_PAD)) * 2;
+}
+
+LLMX_EXPORT int llmx_attention_tiled_fits(int heads, int kv_heads, int D, int V, int maps) {
+    if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || heads / kv_heads > TL_ROWS || (maps != 1 && maps != 2)) return 0;
     if (D <= 0 || V <= 0 || D % 16 || V % 16 || D > 256 || V > 256) return 0;
-    const size_t smem = ((size_t)TL_ROWS * (D + TL_PAD) + 2 * (size_t)TL_KEYS * (D + V + TL_PAD)) * 2;
-    return smem <= 200 * 1024;
+    return tiled_smem(D, V, maps) <= 200 * 1024;
 }
 
 // The tiled form: q [rows, heads, D], out [rows, heads, V] and the cache bfloat16; the step's row ranges and histories
@@ -971,34 +1111,39 @@ LLMX_EXPORT int llmx_attention_tiled_fits(int heads, int kv_heads, int D, int V)
 LLMX_EXPORT int llmx_attention_tiled(const void* q, const void* cache, void* out, const int* row_start, const int* row_count,
                                      const int* history, const int* block_tables, int table_stride, int rows, int requests,
                                      int heads, int kv_heads, int D, int V, int page_size, int window, int chunk, float scale,
-                                     float softcap, const float* sink, int sink_mode, const float* vfreq, int v_neighbours,
-                                     cudaStream_t stream) {
+                                     float softcap, const float* sink, int sink_mode, const float* vfreq, int v_neighbours, int maps,
+                                     float factor, float out_factor, float eps, const float* gate, int gate_stride, cudaStream_t stream) {
     if (rows <= 0 || requests <= 0) return 0;
-    if (sink_mode < 0 || sink_mode > 2 || (sink_mode == 1 && sink == nullptr)) return LLMX_ERR_BAD_ARGUMENT;
-    const AttnExtras extras{softcap, sink, sink_mode, vfreq, v_neighbours};
-    if (!llmx_attention_tiled_fits(heads, kv_heads, D, V) || kv_heads > 65535) return LLMX_ERR_UNSUPPORTED;
+    const AttnExtras extras{softcap, sink, sink_mode, vfreq, v_neighbours, maps, factor, out_factor, eps, gate, gate_stride};
+    if (!extras_fit(extras, heads, kv_heads, V)) return LLMX_ERR_BAD_ARGUMENT;
+    if (!llmx_attention_tiled_fits(heads, kv_heads, D, V, maps) || kv_heads > 65535) return LLMX_ERR_UNSUPPORTED;
     int r_pad = 1;
-    while (r_pad < heads / kv_heads) r_pad *= 2;
-    const int tok = TL_ROWS / r_pad;
+    while (r_pad < heads / kv_heads / maps) r_pad *= 2;
+    const int tok = TL_ROWS / maps / r_pad;
     dim3 grid((rows + tok - 1) / tok + requests, kv_heads);
-    const size_t smem = ((size_t)TL_ROWS * (D + TL_PAD) + 2 * (size_t)TL_KEYS * (D + V + TL_PAD)) * 2;
-#define LLMX_TILED(VN)                                                                                                   \
+    const size_t smem = tiled_smem(D, V, maps);
+#define LLMX_TILED(VN, M)                                                                                                   \
     do {                                                                                                                  \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(attention_tiled_kernel<VN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        launch_kernel(attention_tiled_kernel<VN>, dim3(grid), dim3(128), smem, stream, (const __nv_bfloat16*)q,          \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(attention_tiled_kernel<VN, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        launch_kernel(attention_tiled_kernel<VN, M>, dim3(grid), dim3(128), smem, stream, (const __nv_bfloat16*)q,          \
                       (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, row_start, row_count, history, block_tables,    \
                       table_stride, requests, heads, kv_heads, D, V, page_size, window, chunk, scale, r_pad, extras);   \
         return launch_status();                                                                                           \
     } while (0)
-    if (V <= 64) LLMX_TILED(8);
-    if (V <= 128) LLMX_TILED(16);
-    LLMX_TILED(32);
+    if (maps == 2) {
+        if (V <= 64) LLMX_TILED(8, 2);
+        if (V <= 128) LLMX_TILED(16, 2);
+        LLMX_TILED(32, 2);
+    }
+    if (V <= 64) LLMX_TILED(8, 1);
+    if (V <= 128) LLMX_TILED(16, 1);
+    LLMX_TILED(32, 1);
 #undef LLMX_TILED
 }
 
 // Whether the staged form takes these types and sizes.
-LLMX_EXPORT int llmx_attention_staged_fits(int q_dtype, int cache_dtype, int heads, int kv_heads, int D, int V) {
-    return staged_tile(q_dtype, cache_dtype, heads, kv_heads, D, V, nullptr) > 0;
+LLMX_EXPORT int llmx_attention_staged_fits(int q_dtype, int cache_dtype, int heads, int kv_heads, int D, int V, int maps) {
+    return staged_tile(q_dtype, cache_dtype, heads, kv_heads, D, V, maps, nullptr) > 0;
 }
 
 // The staged form with its merge: arguments as `llmx_attention_split`; `partial` float32 [rows, heads, splits, V + 2] is
@@ -1007,14 +1152,15 @@ LLMX_EXPORT int llmx_attention_staged(const void* q, int q_dtype, const void* ca
                                       const int* row_request, const int* positions, const int* block_tables, int table_stride,
                                       int rows, int heads, int kv_heads, int D, int V, int page_size, int window, int chunk,
                                       float scale, int splits, float* partial, float softcap, const float* sink, int sink_mode,
-                                      const float* vfreq, int v_neighbours, cudaStream_t stream) {
+                                      const float* vfreq, int v_neighbours, int maps, float factor, float out_factor, float eps,
+                                      const float* gate, int gate_stride, cudaStream_t stream) {
     if (rows <= 0) return 0;
     size_t smem = 0;
-    const int tk = staged_tile(q_dtype, cache_dtype, heads, kv_heads, D, V, &smem);
+    const int tk = staged_tile(q_dtype, cache_dtype, heads, kv_heads, D, V, maps, &smem);
     if (tk == 0 || kv_heads > 65535 || ((uintptr_t)cache & 15)) return LLMX_ERR_UNSUPPORTED;
     if (splits < 1 || splits > 64 || partial == nullptr || page_size <= 0) return LLMX_ERR_BAD_ARGUMENT;
-    if (sink_mode < 0 || sink_mode > 2 || (sink_mode == 1 && sink == nullptr) || (vfreq != nullptr && V % 2)) return LLMX_ERR_BAD_ARGUMENT;
-    const AttnExtras extras{softcap, sink, sink_mode, vfreq, v_neighbours};
+    const AttnExtras extras{softcap, sink, sink_mode, vfreq, v_neighbours, maps, factor, out_factor, eps, gate, gate_stride};
+    if (!extras_fit(extras, heads, kv_heads, V)) return LLMX_ERR_BAD_ARGUMENT;
     const dim3 grid(rows, kv_heads, splits);
     const int hpw = (heads / kv_heads + 3) / 4;
 #define LLMX_STAGED(T, H, VL)                                                                                              \
@@ -1022,7 +1168,7 @@ LLMX_EXPORT int llmx_attention_staged(const void* q, int q_dtype, const void* ca
         if (smem > 48 * 1024) cudaFuncSetAttribute(attention_staged_kernel<T, H, VL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         launch_kernel(attention_staged_kernel<T, H, VL>, grid, dim3(128), smem, stream, (const T*)q, (const T*)cache, row_request, \
                       positions, block_tables, table_stride, heads, kv_heads, D, V, page_size, window, chunk, scale, splits, tk, \
-                      softcap, partial);                                                                                    \
+                      softcap, maps, partial);                                                                                    \
     } while (0)
 #define LLMX_STAGED_T(T)                                                                                                   \
     do {                                                                                                                    \
@@ -1042,10 +1188,5 @@ LLMX_EXPORT int llmx_attention_staged(const void* q, int q_dtype, const void* ca
 #undef LLMX_STAGED
     int status = launch_status();
     if (status) return status;
-    const int items = rows * heads;
-    if (q_dtype == LLMX_BF16)
-        launch_kernel(attention_merge_kernel<__nv_bfloat16>, dim3((items + 3) / 4), dim3(128), (size_t)4 * V * sizeof(float), stream, (const float*)partial, (__nv_bfloat16*)out, items, V, splits, heads, positions, extras);
-    else
-        launch_kernel(attention_merge_kernel<float>, dim3((items + 3) / 4), dim3(128), (size_t)4 * V * sizeof(float), stream, (const float*)partial, (float*)out, items, V, splits, heads, positions, extras);
-    return launch_status();
+    return launch_merge(partial, out, q_dtype, rows, heads, V, splits, positions, extras, stream);
 }

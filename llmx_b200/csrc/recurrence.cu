@@ -9,6 +9,8 @@
 // Two more forms share the code.  The scaled form (a selective state space): a_t a gate per row and head,
 // u_t = beta_t * v_t (beta the row's step size), and o_t += skip_h * v_t.  The delta rule with a decay per key
 // channel: S <- diag(g_t) S with g_t [D] per row and head, then u_t = beta_t * (v_t - S^T k_t), S <- S + k_t u_t^T.
+// Gated linear attention is that without the correction: S <- diag(g_t) S + k_t v_t^T; its gates are made by
+// `llmx_channel_decay`.
 // Column j of S (the D values that meet v's entry j) never meets another column, so the work is cut by columns:
 // a few threads own one column, each holding a share of its values in registers for all of the request's rows;
 // the two dot products are sums over a lane's values and then over the column's lanes by shuffles.  A block holds
@@ -32,8 +34,11 @@
 namespace {
 constexpr int REC_THREADS = 128;
 // What a row does to the state: a constant decay per head; the delta rule with one gate per row and head; a gate per
-// row and head with the input scaled by beta and a skip term; the delta rule with a gate per row, head and key channel.
-constexpr int M_CONST = 0, M_DELTA = 1, M_SCALED = 2, M_DELTA_VEC = 3;
+// row and head with the input scaled by beta and a skip term; the delta rule with a gate per row, head and key channel;
+// such a gate alone.
+constexpr int M_CONST = 0, M_DELTA = 1, M_SCALED = 2, M_DELTA_VEC = 3, M_VEC = 4;
+constexpr bool has_channel_gate(int mode) { return mode == M_DELTA_VEC || mode == M_VEC; }
+constexpr bool has_beta(int mode) { return mode != M_CONST && mode != M_VEC; }
 
 // The form for steps of a row or a few: LANES (8) threads share one column of the state, each holding PER of its D
 // values (D <= LANES * PER), so a sum over the lanes is three shuffle steps; a block of 128 threads owns 16 columns of
@@ -69,7 +74,7 @@ recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         const int d = lane + i * LANES;
         S[i] = (!fresh && d < D) ? sin_[d] : 0.0f;
     }
-    constexpr bool VEC = MODE == M_DELTA_VEC;
+    constexpr bool VEC = has_channel_gate(MODE);
     constexpr int GP = VEC ? PER : 1;
     const float dec = MODE == M_CONST ? decay[h] : VEC ? 1.0f : 0.0f;
     const float sk = MODE == M_SCALED && skip != nullptr ? skip[h] : 0.0f;
@@ -87,7 +92,7 @@ recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         }
         fu = v[row * v_stride + (size_t)h * V + j];
         if (MODE == M_DELTA || MODE == M_SCALED) fa = gate[row * gate_stride + h];
-        if (MODE != M_CONST) fb = beta[row * beta_stride + h];
+        if (has_beta(MODE)) fb = beta[row * beta_stride + h];
         if (VEC) {
             const float* gp = gate + row * gate_stride + (size_t)h * D;
 #pragma unroll
@@ -105,7 +110,7 @@ recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 #pragma unroll
             for (int i = 0; i < PER; ++i) S[i] *= gg[i < GP ? i : 0];
         }
-        if (MODE == M_DELTA || VEC) {
+        if (MODE == M_DELTA || MODE == M_DELTA_VEC) {
             float dot = 0.0f;
 #pragma unroll
             for (int i = 0; i < PER; ++i) dot = fmaf(S[i], kk[i], dot);
@@ -186,7 +191,7 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float stage[];   // [2][WIDE_CH][row_floats]: q (Dp), k (Dp), [gates per channel (Dp)], v (8 columns), gate, beta, pad
-    constexpr bool VEC = MODE == M_DELTA_VEC;
+    constexpr bool VEC = has_channel_gate(MODE);
     constexpr int NV = VEC ? 3 : 2;                  // vectors of D values a row brings
     const int Dp = PER * 32;                         // a row's q and k padded to the lanes' runs (the pad is never written: zeros are read by the guard)
     const int row_floats = NV * Dp + WIDE_COLS + 4;  // a multiple of 4: every row starts on 16 bytes
@@ -247,7 +252,7 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
                 ++t;
             }
         }
-        if (small_t < rows && (small_e < WIDE_COLS || (small_e == WIDE_COLS ? (MODE == M_DELTA || MODE == M_SCALED) : MODE != M_CONST))) {
+        if (small_t < rows && (small_e < WIDE_COLS || (small_e == WIDE_COLS ? (MODE == M_DELTA || MODE == M_SCALED) : has_beta(MODE)))) {
             const size_t row = (size_t)(a0 + t0 + small_t);
             const float* src = small_e < WIDE_COLS ? v + row * v_stride + (size_t)h * V + min(first_col + small_e, V - 1)
                              : small_e == WIDE_COLS ? gate + row * gate_stride + h : beta + row * beta_stride + h;
@@ -278,7 +283,7 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
                 for (int i = 0; i < PER; ++i) S[i] *= gg[i];     // past D: S stays zero whatever the pad holds... the guard reads zeros there
             }
             if (MODE == M_DELTA || MODE == M_SCALED) a = rowp[NV * Dp + WIDE_COLS];
-            if (MODE == M_DELTA || VEC) {
+            if (MODE == M_DELTA || MODE == M_DELTA_VEC) {
                 float dot = 0.0f;
 #pragma unroll
                 for (int i = 0; i < PER; ++i) dot = fmaf(S[i], kk[i], dot);
@@ -393,6 +398,48 @@ conv_prepare_kernel(const float* __restrict__ proj, int stride, int first, int c
     }
 }
 
+// Decays per key channel through a low-rank pair, in 32-bit: z = low W2^T + bias, decay = sigmoid(z)^(1 / tau); `low` is the
+// pair's inner values (a run of columns of the projections), `w2t` W2 transposed [rank][channels].  In passing the same
+// channels of q (columns q_off .. of the projections) are multiplied by `q_factor`.  A thread a channel, DECAY_ROWS rows.
+constexpr int DECAY_ROWS = 8, DECAY_THREADS = 128, DECAY_RANK = 64;
+
+__global__ void __launch_bounds__(DECAY_THREADS)
+channel_decay_kernel(float* __restrict__ proj, int stride, int rows, int low_off, int rank, const float* __restrict__ w2t,
+                     const float* __restrict__ bias, float inv_tau, float* __restrict__ decay, int channels, int q_off, float q_factor) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float low[DECAY_RANK][DECAY_ROWS];
+    const int c = blockIdx.x * DECAY_THREADS + threadIdx.x;
+    const int r0 = blockIdx.y * DECAY_ROWS, n = min(DECAY_ROWS, rows - r0);
+    const float b = bias && c < channels ? bias[c] : 0.0f;
+    float z[DECAY_ROWS];
+#pragma unroll
+    for (int r = 0; r < DECAY_ROWS; ++r) z[r] = b;
+    for (int k0 = 0; k0 < rank; k0 += DECAY_RANK) {
+        const int kn = min(DECAY_RANK, rank - k0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < kn * DECAY_ROWS; i += DECAY_THREADS) {
+            const int r = i / kn, k = i - r * kn;
+            low[k][r] = r < n ? proj[(size_t)(r0 + r) * stride + low_off + k0 + k] : 0.0f;
+        }
+        __syncthreads();
+        if (c < channels)
+            for (int k = 0; k < kn; ++k) {
+                const float w = w2t[(size_t)(k0 + k) * channels + c];
+#pragma unroll
+                for (int r = 0; r < DECAY_ROWS; ++r) z[r] = fmaf(low[k][r], w, z[r]);
+            }
+    }
+    if (c >= channels) return;
+#pragma unroll
+    for (int r = 0; r < DECAY_ROWS; ++r) {
+        if (r >= n) break;
+        const float log_sigmoid = fminf(z[r], 0.0f) - log1pf(expf(-fabsf(z[r])));
+        decay[(size_t)(r0 + r) * channels + c] = expf(log_sigmoid * inv_tau);
+        if (q_factor != 1.0f) proj[(size_t)(r0 + r) * stride + q_off + c] *= q_factor;
+    }
+}
+
 template <int MODE>
 int launch_recurrence(int D, bool wide, int requests, cudaStream_t stream, const float* q, const float* k, const float* v,
                       int q_stride, int k_stride, int v_stride, const float* decay, const float* gate, const float* beta,
@@ -413,7 +460,7 @@ int launch_recurrence(int D, bool wide, int requests, cudaStream_t stream, const
     do {                                                                                                                  \
         const long long by = (long long)heads * ((V + WIDE_COLS - 1) / WIDE_COLS);                                        \
         if (by > 65535) return LLMX_ERR_UNSUPPORTED;                                                                      \
-        const size_t smem = (size_t)2 * WIDE_CH * ((MODE == M_DELTA_VEC ? 3 : 2) * P * 32 + WIDE_COLS + 4) * sizeof(float);   \
+        const size_t smem = (size_t)2 * WIDE_CH * ((has_channel_gate(MODE) ? 3 : 2) * P * 32 + WIDE_COLS + 4) * sizeof(float);   \
         if (smem > 200 * 1024) return LLMX_ERR_UNSUPPORTED;                                                               \
         if (smem > 48 * 1024)                                                                                             \
             cudaFuncSetAttribute(recurrence_wide_kernel<P, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
@@ -444,7 +491,8 @@ int launch_recurrence(int D, bool wide, int requests, cudaStream_t stream, const
 // q, k [rows, qk_heads * D] and v [rows, heads * V] floats with row strides of their own (they may lie inside one wider
 // matrix).  `mode` 0: a constant `decay` [heads].  1: the delta rule, `gate` and `beta` [rows, .] (row strides
 // `gate_stride`, `beta_stride`, entry h).  2: the scaled form, a = gate, u = beta * v, out += skip_h * v (`skip` [heads]
-// or null).  3: the delta rule with `gate` [rows, heads * D] (entry h * D + d), a decay per key channel.  `state`: the
+// or null).  3: the delta rule with `gate` [rows, heads * D] (entry h * D + d), a decay per key channel.  4: `gate` as in 3,
+// u = v (gated linear attention; no beta).  `state`: the
 // slots' storage, `slot_floats` apart, the recurrence's [H][V][D] at its start; out [rows, heads * V] floats.  The
 // metadata arrays are the step's, on the device.
 LLMX_EXPORT int llmx_linear_recurrence(const float* q, const float* k, const float* v, int q_stride, int k_stride,
@@ -456,7 +504,8 @@ LLMX_EXPORT int llmx_linear_recurrence(const float* q, const float* k, const flo
                                        cudaStream_t stream) {
     if (requests <= 0) return 0;
     if (heads <= 0 || qk_heads <= 0 || heads % qk_heads || D <= 0 || V <= 0 || D > 512) return LLMX_ERR_UNSUPPORTED;
-    if (mode < 0 || mode > 3 || (mode == M_CONST ? decay == nullptr : (gate == nullptr || beta == nullptr))) return LLMX_ERR_BAD_ARGUMENT;
+    if (mode < 0 || mode > 4 || (mode == M_CONST ? decay == nullptr : (gate == nullptr || (beta == nullptr && has_beta(mode)))))
+        return LLMX_ERR_BAD_ARGUMENT;
     const bool wide = max_rows > 8;            // `max_rows`: the most rows one request brings (a matter of speed only)
 #define LLMX_MODE(M)                                                                                                      \
     return launch_recurrence<M>(D, wide, requests, stream, q, k, v, q_stride, k_stride, v_stride, decay, gate, beta,      \
@@ -465,7 +514,8 @@ LLMX_EXPORT int llmx_linear_recurrence(const float* q, const float* k, const flo
     if (mode == M_CONST) LLMX_MODE(M_CONST);
     if (mode == M_DELTA) LLMX_MODE(M_DELTA);
     if (mode == M_SCALED) LLMX_MODE(M_SCALED);
-    LLMX_MODE(M_DELTA_VEC);
+    if (mode == M_DELTA_VEC) LLMX_MODE(M_DELTA_VEC);
+    LLMX_MODE(M_VEC);
 #undef LLMX_MODE
 }
 
@@ -494,5 +544,21 @@ LLMX_EXPORT int llmx_conv_prepare(const float* proj, int stride, int first, int 
                   q_channels, k_channels, taps_w, taps_b, taps, ready, a_log, dt_bias, b_off, a_off, gate_kind, decay_in,
                   decay_stride, gates, gates_stride, heads, D, q_factor, state, slot_floats, conv_off, row_request,
                   row_start, row_count, history, slot_in, slot_out, rows);
+    return launch_status();
+}
+
+// proj [rows, stride]: the pair's inner values in columns low_off .. low_off + rank - 1, q in columns q_off .. q_off + channels
+// - 1 (multiplied in place by q_factor; the two runs must not overlap); w2t [rank, channels], bias [channels] or null;
+// decay [rows, channels] = sigmoid(low w2t + bias)^inv_tau.
+LLMX_EXPORT int llmx_channel_decay(float* proj, int stride, int rows, int low_off, int rank, const float* w2t, const float* bias,
+                                   float inv_tau, float* decay, int channels, int q_off, float q_factor, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (rank < 1 || channels < 1 || low_off < 0 || q_off < 0 || low_off + rank > stride || q_off + channels > stride ||
+        (low_off < q_off + channels && q_off < low_off + rank) || w2t == nullptr)
+        return LLMX_ERR_BAD_ARGUMENT;
+    const long long by = ((long long)rows + DECAY_ROWS - 1) / DECAY_ROWS;
+    if (by > 65535) return LLMX_ERR_UNSUPPORTED;
+    launch_kernel(channel_decay_kernel, dim3((channels + DECAY_THREADS - 1) / DECAY_THREADS, (unsigned)by), dim3(DECAY_THREADS), 0, stream,
+                  proj, stride, rows, low_off, rank, w2t, bias, inv_tau, decay, channels, q_off, q_factor);
     return launch_status();
 }

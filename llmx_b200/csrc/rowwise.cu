@@ -717,6 +717,104 @@ LLMX_EXPORT int llmx_layernorm(const float* x, const float* w, void* y, int out_
 }
 
 // ---------------------------------------------------------------------------
+// The RMS norm after a sublayer: z = y + in_bias; x += z / sqrt(mean(z^2) + eps) * w, all 32-bit; the new row of the stream
+// also goes to `copy` in the type the next products read, and blocks of their own clear `zero` (what those products add
+// into).  Without `y` only the copy and the clearing are made.  One block a row; VEC4: rows read in pieces of four values
+// that stay in registers between the two passes.
+// ---------------------------------------------------------------------------
+template <typename CopyT, bool VEC4>
+__global__ void rmsnorm_add_kernel(const float* __restrict__ y, const float* __restrict__ in_bias, const float* __restrict__ w,
+                                   float* __restrict__ x, CopyT* __restrict__ copy, int rows, int width, float eps,
+                                   float* __restrict__ zero, long long zero_count) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int r = blockIdx.x;
+    if (r >= rows) {
+        float4* z = reinterpret_cast<float4*>(zero);
+        const long long n4 = zero_count >> 2, blocks = gridDim.x - rows;
+        for (long long i = (long long)(r - rows) * blockDim.x + threadIdx.x; i < n4; i += blocks * blockDim.x)
+            z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        return;
+    }
+    float* xr = x + (size_t)r * width;
+    CopyT* cr = copy ? copy + (size_t)r * width : nullptr;
+    const float* yr = y ? y + (size_t)r * width : nullptr;
+    if constexpr (VEC4) {
+        const int n4 = width >> 2;
+        float4 v[NORM_VEC_MAX];
+        float s = 0.0f;
+        if (yr) {
+#pragma unroll
+            for (int k = 0; k < NORM_VEC_MAX; ++k) {
+                const int i = threadIdx.x + k * blockDim.x;
+                v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i >= n4) continue;
+                v[k] = read4(yr + 4 * i);
+                if (in_bias) {
+                    const float4 b = read4(in_bias + 4 * i);
+                    v[k] = make_float4(v[k].x + b.x, v[k].y + b.y, v[k].z + b.z, v[k].w + b.w);
+                }
+                s = fmaf(v[k].x, v[k].x, s);
+                s = fmaf(v[k].y, v[k].y, s);
+                s = fmaf(v[k].z, v[k].z, s);
+                s = fmaf(v[k].w, v[k].w, s);
+            }
+        }
+        const float rr = yr ? 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps) : 0.0f;
+#pragma unroll
+        for (int k = 0; k < NORM_VEC_MAX; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i >= n4) continue;
+            float4 t = read4(xr + 4 * i);
+            if (yr) {
+                const float4 ww = read4(w + 4 * i);
+                t = make_float4(fmaf(v[k].x * rr, ww.x, t.x), fmaf(v[k].y * rr, ww.y, t.y), fmaf(v[k].z * rr, ww.z, t.z),
+                                fmaf(v[k].w * rr, ww.w, t.w));
+                store4(xr + 4 * i, t.x, t.y, t.z, t.w);
+            }
+            if (cr) store4(cr + 4 * i, t.x, t.y, t.z, t.w);
+        }
+    } else {
+        float s = 0.0f;
+        if (yr)
+            for (int i = threadIdx.x; i < width; i += blockDim.x) {
+                const float z = yr[i] + (in_bias ? in_bias[i] : 0.0f);
+                s = fmaf(z, z, s);
+            }
+        const float rr = yr ? 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps) : 0.0f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            float t = xr[i];
+            if (yr) {
+                t = fmaf((yr[i] + (in_bias ? in_bias[i] : 0.0f)) * rr, w[i], t);
+                xr[i] = t;
+            }
+            if (cr) cr[i] = from_float<CopyT>(t);
+        }
+    }
+}
+
+LLMX_EXPORT int llmx_rmsnorm_add(const float* y, const float* in_bias, const float* w, float* x, void* copy, int copy_dtype, int rows,
+                                 int width, float eps, float* zero, long long zero_count, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (width <= 0 || (y != nullptr && w == nullptr)) return LLMX_ERR_BAD_ARGUMENT;
+    if (zero && (zero_count % 4 || ((uintptr_t)zero & 15))) return LLMX_ERR_BAD_ARGUMENT;
+    const bool vec4 = width % 4 == 0 && width <= 4 * NORM_VEC_MAX * 256 &&
+                      !(((uintptr_t)y | (uintptr_t)in_bias | (uintptr_t)w | (uintptr_t)x | (uintptr_t)copy) & 15);
+    const int threads = vec4 ? norm_threads(width) : 256;
+    long long zero_blocks = zero ? (zero_count / 4 + 4 * threads - 1) / (4 * threads) : 0;
+    zero_blocks = zero_blocks > 1024 ? 1024 : zero_blocks;
+    const dim3 grid((unsigned)(rows + zero_blocks));
+#define LLMX_RADD(T, R) launch_kernel(rmsnorm_add_kernel<T, R>, grid, dim3(threads), 0, stream, y, in_bias, w, x, (T*)copy, rows, width, eps, zero, zero_count)
+    if (copy_dtype == LLMX_BF16 && vec4) LLMX_RADD(__nv_bfloat16, true);
+    else if (copy_dtype == LLMX_BF16) LLMX_RADD(__nv_bfloat16, false);
+    else if (vec4) LLMX_RADD(float, true);
+    else LLMX_RADD(float, false);
+#undef LLMX_RADD
+    return launch_status();
+}
+
+// ---------------------------------------------------------------------------
 // A gate on rows: o[r, c] *= sigmoid(gate[r, c]) in 32-bit, o of the path's type in place; `gate` is float and has a
 // row stride of its own (it lies inside a wider product's output).
 // ---------------------------------------------------------------------------

@@ -291,10 +291,13 @@ class Model:
         x0 = None
         if any(s.add_embedding for s in self.order):
             x0 = x.clone()
-        for s in self.order:
+        for n, s in enumerate(self.order):
             if s.add_embedding:
                 from .. import ops
                 ops.add_(x, x0)
+            # The block that reads the stream next (None when something else changes it first): a block may prepare its input.
+            then = self.order[n + 1] if n + 1 < len(self.order) else None
+            step.extras["next_block"] = self.blocks[then.block] if then is not None and not then.add_embedding else None
             self.blocks[s.block].forward(x, step, s.cache_entry, s.write_cache)
         if wanted == 0:
             return None

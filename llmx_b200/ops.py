@@ -107,6 +107,8 @@ _SIGNATURES = {
     ("rowwise", "llmx_clamped_glu"): [_p, _p, _i, _i, _i, _f, _f, _p],
     ("rowwise", "llmx_silu_columns"): [_p, _i, _i, _i, _i, _p],
     ("rowwise", "llmx_gated_rmsnorm"): [_p, _p, _i, _p, _i, _p, _i, _i, _i, _i, _f, _i, _i, _p],
+    ("rowwise", "llmx_rmsnorm_add"): [_p, _p, _p, _p, _p, _i, _i, _i, _f, _p, ctypes.c_longlong, _p],
+    ("recurrence", "llmx_channel_decay"): [_p, _i, _i, _i, _i, _p, _p, _f, _p, _i, _i, _f, _p],
     ("rowwise", "llmx_pair_norm_add"): [_p, _p, _p, _p, _p, _i, _i, _f, _f, _p],
     ("rowwise", "llmx_add"): [_p, _p, ctypes.c_longlong, _p],
     ("recurrence", "llmx_linear_recurrence"): [_p, _p, _p, _i, _i, _i, _i, _p, _p, _p, _i, _i, _p, _p, ctypes.c_longlong, _p, _p,
@@ -115,15 +117,15 @@ _SIGNATURES = {
                                           _p, ctypes.c_longlong, ctypes.c_longlong, _p, _p, _p, _p, _p, _p, _i, _i, _p],
     ("attention_split", "llmx_qk_norm_rope_write"): [_p, _i, _p, _p, _f, _p, _i, _p, _p, _p, _i, _p, _i, _i, _i, _i, _i, _i, _i, _p],
     ("attention_split", "llmx_qkv_finish"): [_p, _i, _p, _p, _i, _p, ctypes.c_longlong, ctypes.c_longlong, _p, _p, _p, _p, _p, _p, _p, _p, _i,
-                                             _f, _p, _i, _i, _p, _p, _p, _i, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p],
+                                             _f, _p, _i, _i, _p, _p, _p, _i, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p],
     ("attention_split", "llmx_attention_split"): [_p, _i, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p,
-                                                  _f, _p, _i, _p, _i, _p],
+                                                  _f, _p, _i, _p, _i, _i, _f, _f, _f, _p, _i, _p],
     ("attention_split", "llmx_attention_staged"): [_p, _i, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p,
-                                                   _f, _p, _i, _p, _i, _p],
-    ("attention_split", "llmx_attention_staged_fits"): [_i, _i, _i, _i, _i, _i],
-    ("attention_split", "llmx_attention_tiled_fits"): [_i, _i, _i, _i],
+                                                   _f, _p, _i, _p, _i, _i, _f, _f, _f, _p, _i, _p],
+    ("attention_split", "llmx_attention_staged_fits"): [_i, _i, _i, _i, _i, _i, _i],
+    ("attention_split", "llmx_attention_tiled_fits"): [_i, _i, _i, _i, _i],
     ("attention_split", "llmx_attention_tiled"): [_p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f,
-                                                  _f, _p, _i, _p, _i, _p],
+                                                  _f, _p, _i, _p, _i, _i, _f, _f, _f, _p, _i, _p],
     ("moe", "llmx_moe_route"): [_p, _p, _i, _i, _i, _i, _p, _p, _p, _i, _p],
     ("moe", "llmx_moe_product_few"): [_p, _i, _p, _p, _p, _i, _i, _i, _i, _p, _i, _i, _i, _i, _i, _f, _f, _p],
     ("moe", "llmx_moe_product"): [_p, _i, _p, _i, _p, _p, _p, _i, _i, _p, _i, _i, _i, _i, _i, _f, _f, _i, _p],
@@ -442,6 +444,25 @@ def layernorm_add_(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor
     return residual
 
 
+def rmsnorm_add_(x: torch.Tensor, y: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float,
+                 in_bias: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None, zero: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += z / sqrt(mean(z^2) + eps) * weight row by row, z = y + in_bias, all float32; then `copy` (the type the products that
+    follow read) takes the new x, and the float32 buffer `zero` is cleared by the same launch.  Without y: copy and clearing
+    alone."""
+    _cuda(x, y, weight, in_bias, copy, zero)
+    rows, width = x.shape
+    _need(x.dtype == torch.float32 and (y is None or (y.dtype == torch.float32 and tuple(y.shape) == (rows, width) and weight is not None)),
+          "rmsnorm_add: float32 tensors of one shape and a weight")
+    for t in (weight, in_bias):
+        _need(t is None or (t.dtype == torch.float32 and t.numel() == width), "rmsnorm_add: float32 vectors of the row's width")
+    _need(copy is None or tuple(copy.shape) == (rows, width), "rmsnorm_add: the copy has the rows' shape")
+    _need(zero is None or (zero.dtype == torch.float32 and zero.numel() % 4 == 0), "rmsnorm_add: a float32 buffer of whole 16-byte pieces to clear")
+    _check(_fn("rowwise", "llmx_rmsnorm_add")(_ptr(y), _ptr(in_bias), _ptr(weight), _ptr(x), _ptr(copy), F32 if copy is None else _code(copy),
+                                              rows, width, float(eps), _ptr(zero), 0 if zero is None else zero.numel(), _stream()),
+           "rmsnorm_add")
+    return x
+
+
 def add_bias_(x: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
     """x[r, :] += bias; float32."""
     _cuda(x, bias)
@@ -610,6 +631,7 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: 
       "delta"          a = gate, u = beta (v - a S^T k); gate, beta [rows, heads] (views)
       "scaled"         a = gate, u = beta v, o += skip_h v; gate, beta [rows, heads], skip [heads] or None
       "delta_channel"  S <- diag(gate) S first, gate [rows, heads * D]; then u = beta (v - S^T k), S <- S + k u^T
+      "channel"        S <- diag(gate) S + k v^T, gate [rows, heads * D] (no beta)
     q, k [rows, qk_heads * D], v [rows, heads * V]: float32 views whose rows may be strided.  state [slots, floats]: the
     recurrence's values first, [H][V][D].  `step`: the StepBatch (row ranges, histories and slots are read on the device)."""
     rows = q.shape[0]
@@ -621,15 +643,15 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: 
     _need(out.dtype == torch.float32 and tuple(out.shape) == (rows, heads * value_dim), "recurrence: output shape does not fit")
     if form is None:
         form = "delta" if gate is not None else "decay"
-    _need(form in ("decay", "delta", "scaled", "delta_channel"), "recurrence: unknown form")
-    mode = ("decay", "delta", "scaled", "delta_channel").index(form)
+    _need(form in ("decay", "delta", "scaled", "delta_channel", "channel"), "recurrence: unknown form")
+    mode = ("decay", "delta", "scaled", "delta_channel", "channel").index(form)
     gs = bs = 0
     if mode == 0:
         _need(decay is not None and decay.dtype == torch.float32 and decay.numel() == heads and gate is None, "recurrence: decay float32 [heads]")
     else:
-        _need(gate is not None and beta is not None and decay is None, "recurrence: this form takes gate and beta and no constant decay")
-        gs, bs = _strided_rows(gate, "recurrence gate"), _strided_rows(beta, "recurrence beta")
-        _need(tuple(gate.shape) == (rows, heads * key_dim if mode == 3 else heads) and tuple(beta.shape) == (rows, heads),
+        _need(gate is not None and (beta is None) == (mode == 4) and decay is None, "recurrence: this form takes gate and beta (\"channel\": gate alone) and no constant decay")
+        gs, bs = _strided_rows(gate, "recurrence gate"), 0 if beta is None else _strided_rows(beta, "recurrence beta")
+        _need(tuple(gate.shape) == (rows, heads * key_dim if mode >= 3 else heads) and (beta is None or tuple(beta.shape) == (rows, heads)),
               "recurrence: gate [rows, heads] (or [rows, heads * D] per key channel) and beta [rows, heads]")
     if skip is not None:
         _need(mode == 2 and skip.dtype == torch.float32 and skip.numel() == heads, "recurrence: skip float32 [heads], scaled form only")
@@ -639,6 +661,23 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: 
         _ptr(step.state_slots_out), _ptr(out), step.requests, heads, qk_heads, key_dim, value_dim, int(step.max_row_count),
         _stream()), "linear_recurrence")
     return out
+
+
+def channel_decay_(proj: torch.Tensor, low_off: int, w2t: torch.Tensor, bias: Optional[torch.Tensor], tau: float,
+                   decay: torch.Tensor, q_off: int, q_factor: float) -> torch.Tensor:
+    """decay [rows, channels] = sigmoid(low w2t + bias)^(1 / tau), 32-bit; `low`: columns low_off .. of the projections `proj`
+    (float32 [rows, width]), w2t float32 [rank, channels].  Columns q_off .. q_off + channels - 1 of `proj` are multiplied by
+    `q_factor` in place."""
+    _cuda(proj, w2t, bias, decay)
+    rows = proj.shape[0]
+    rank, channels = w2t.shape
+    _need(proj.dtype == torch.float32 and proj.dim() == 2 and w2t.dtype == torch.float32 and decay.dtype == torch.float32
+          and tuple(decay.shape) == (rows, channels), "channel_decay: float32 projections, weight [rank, channels] and decay [rows, channels]")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == channels), "channel_decay: float32 bias [channels]")
+    _need(0 <= low_off and low_off + rank <= proj.shape[1] and 0 <= q_off and q_off + channels <= proj.shape[1], "channel_decay: columns outside the projections")
+    _check(_fn("recurrence", "llmx_channel_decay")(_ptr(proj), proj.shape[1], rows, int(low_off), rank, _ptr(w2t), _ptr(bias), 1.0 / float(tau),
+                                                   _ptr(decay), channels, int(q_off), float(q_factor), _stream()), "channel_decay")
+    return decay
 
 
 def conv_prepare(proj: torch.Tensor, channels: int, q_channels: int, k_channels: int, taps_w: torch.Tensor,
@@ -714,7 +753,7 @@ def qkv_finish(proj: torch.Tensor, heads: int, kv_heads: int, key_dim: int, valu
                taps_w: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, conv_off: int = 0,
                norm: str = "none", q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
                freq: Optional[torch.Tensor] = None, neighbours: bool = False, rot_mag: float = 1.0,
-               vfreq: Optional[torch.Tensor] = None) -> None:
+               vfreq: Optional[torch.Tensor] = None, maps: int = 1) -> None:
     """The general finishing of a stacked q/k/v product's rows (csrc/attention_split.cu, `QkvFinish`): proj float32 [rows, q
     (heads * D) | k (kv_heads * D) | v (kv_heads * V)] (a view whose rows may be strided; kv_heads 0: queries alone) plus
     `bias` [channels]; a causal filter `taps_w` [channels, taps] per channel whose earlier inputs lie in `state`
@@ -725,15 +764,18 @@ def qkv_finish(proj: torch.Tensor, heads: int, kv_heads: int, key_dim: int, valu
     has planes of keys and of values, [pages, 2, kv_heads, page, D] (D = V), to those.  `step`: the StepBatch.
     `norm` "whole": one RMS norm over all of a row's queries and one over all of its keys, before they are split into
     heads, with weights [heads * D] and [kv_heads * D].  `rot_mag`: a factor on the rotation's cosines and sines.  `vfreq`
-    float32 [V / 2]: the values are rotated too, over all of V, pair m by position * vfreq[m], in the same pairing."""
+    float32 [V / 2]: the values are rotated too, over all of V, pair m by position * vfreq[m], in the same pairing.
+    `maps` n: every query head and every key/value head has n queries or keys (head by head in the product) and the cache
+    rows are n keys and one value."""
     _cuda(bias, taps_w, state, q_weight, k_weight, freq, slots, q_out, cache, vfreq)
     rows = proj.shape[0]
-    channels = (heads + kv_heads) * key_dim + kv_heads * value_dim
+    heads = heads * maps
+    channels = (heads + kv_heads * maps) * key_dim + kv_heads * value_dim
     _need(proj.is_cuda and proj.dtype == torch.float32 and proj.dim() == 2 and proj.shape[1] == channels and proj.stride(1) == 1,
           "qkv_finish: product rows float32 [rows, q | k | v]")
     _need(tuple(q_out.shape) == (rows, heads * key_dim) and rows == step.rows, "qkv_finish: q_out shape or the step's rows do not fit")
     _need(norm in ("none", "before", "after", "whole"), "qkv_finish: norm is none, before, after or whole")
-    qn, kn = (heads * key_dim, kv_heads * key_dim) if norm == "whole" else (key_dim, key_dim)
+    qn, kn = (heads * key_dim, kv_heads * maps * key_dim) if norm == "whole" else (key_dim, key_dim)
     for t, n in ((bias, channels), (q_weight, qn), (k_weight, kn)):
         _need(t is None or (t.dtype == torch.float32 and t.numel() == n), "qkv_finish: float32 bias [channels], norm weights [D] (whole: [heads * D])")
     _need(vfreq is None or (vfreq.dtype == torch.float32 and 2 * vfreq.numel() == value_dim), "qkv_finish: value frequencies float32 [V / 2]")
@@ -746,8 +788,8 @@ def qkv_finish(proj: torch.Tensor, heads: int, kv_heads: int, key_dim: int, valu
               and conv_off + (taps - 1) * channels <= state.shape[1], "qkv_finish: state slots too small for the filter's inputs")
     if kv_heads:
         _need(cache is not None and slots is not None and cache.dim() == 5 and cache.shape[2] == kv_heads and cache.is_contiguous()
-              and ((cache.shape[1] == 1 and cache.shape[4] == key_dim + value_dim)
-                   or (cache.shape[1] == 2 and key_dim == value_dim and cache.shape[4] == key_dim))
+              and ((cache.shape[1] == 1 and cache.shape[4] == maps * key_dim + value_dim)
+                   or (maps == 1 and cache.shape[1] == 2 and key_dim == value_dim and cache.shape[4] == key_dim))
               and slots.dtype == torch.int32 and slots.numel() >= rows, "qkv_finish: cache layout or slots do not fit")
     _need(freq is None or (freq.dtype == torch.float32 and 2 * freq.numel() <= key_dim), "qkv_finish: frequencies float32 [<= D / 2]")
     _check(_fn("attention_split", "llmx_qkv_finish")(
@@ -757,7 +799,7 @@ def qkv_finish(proj: torch.Tensor, heads: int, kv_heads: int, key_dim: int, valu
         ("none", "before", "after", "whole").index(norm), float(eps), _ptr(freq), 0 if freq is None else freq.numel(), 1 if neighbours else 0,
         _ptr(step.positions), _ptr(slots), _ptr(q_out), _code(q_out), _ptr(cache), _code(cache) if cache is not None else F32, rows,
         step.requests, heads, kv_heads, key_dim, value_dim, cache.shape[3] if cache is not None else 1,
-        cache.shape[1] if cache is not None else 1, float(rot_mag), _ptr(vfreq), _stream()), "qkv_finish")
+        cache.shape[1] if cache is not None else 1, int(maps), float(rot_mag), _ptr(vfreq), _stream()), "qkv_finish")
 
 
 class SoftmaxExtras:
@@ -765,12 +807,29 @@ class SoftmaxExtras:
     `softcap` c > 0: score <- c tanh(score / c) after the scale; `sink`: a float32 tensor [heads] whose exp joins each head's
     denominator (it has no key and no value), or the string "zero" for a sink of 0 (one is added to the denominator);
     `vfreq` float32 [V / 2]: the cached values were rotated by their positions, and a row's output is turned back by its
-    own (`v_neighbours`: pairs (2m, 2m + 1) instead of (m, m + V / 2))."""
+    own (`v_neighbours`: pairs (2m, 2m + 1) instead of (m, m + V / 2)); `difference` = (factor, out_factor, eps): every head
+    has two maps (queries and keys of its own over the same values; q [rows, heads * 2 * D], cache rows [key 1 ; key 2 ; value]),
+    and its output is a1 - factor * a2 over its root mean square (eps inside the root), times out_factor; `gate` float32 [rows,
+    heads], a view whose rows may be strided: head h's output times sigmoid(gate[:, h])."""
 
-    def __init__(self, softcap: Optional[float] = None, sink=None, vfreq: Optional[torch.Tensor] = None, v_neighbours: bool = False):
+    def __init__(self, softcap: Optional[float] = None, sink=None, vfreq: Optional[torch.Tensor] = None, v_neighbours: bool = False,
+                 difference=None, gate: Optional[torch.Tensor] = None):
         self.softcap, self.sink, self.vfreq, self.v_neighbours = softcap, sink, vfreq, bool(v_neighbours)
+        self.difference, self.gate = None if difference is None else tuple(float(x) for x in difference), gate
 
-    def checked(self, heads: int, value_dim: int):
+    @property
+    def maps(self) -> int:
+        return 1 if self.difference is None else 2
+
+    def with_gate(self, gate: torch.Tensor) -> "SoftmaxExtras":
+        return SoftmaxExtras(self.softcap, self.sink, self.vfreq, self.v_neighbours, self.difference, gate)
+
+    def checked(self, heads: int, value_dim: int, rows: int):
+        gate_stride = 0
+        if self.gate is not None:
+            gate_stride = _strided_rows(self.gate, "attention: gate")
+            _need(tuple(self.gate.shape) == (rows, heads), "attention: a gate per row and head")
+        _need(self.difference is None or (self.sink is None and self.vfreq is None), "attention: two maps come without sink and rotated values")
         learned = isinstance(self.sink, torch.Tensor)
         if learned:
             _cuda(self.sink)
@@ -782,7 +841,8 @@ class SoftmaxExtras:
             _need(self.vfreq.dtype == torch.float32 and 2 * self.vfreq.numel() == value_dim, "attention: value frequencies float32 [V / 2]")
         _need(self.softcap is None or self.softcap > 0, "attention: the cap on the scores must be positive")
         return (float(self.softcap or 0.0), _ptr(self.sink if learned else None), 1 if learned else 2 if self.sink == "zero" else 0,
-                _ptr(self.vfreq), 1 if self.v_neighbours else 0)
+                _ptr(self.vfreq), 1 if self.v_neighbours else 0, self.maps, *(self.difference or (0.0, 1.0, 0.0)),
+                ctypes.c_void_p(0 if self.gate is None else self.gate.data_ptr()), gate_stride)
 
 
 NO_EXTRAS = SoftmaxExtras()
@@ -800,19 +860,21 @@ def attention_split(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, row
     values into shared memory once for all heads of the group (a matter of speed: the same sums in another order)."""
     _cuda(q, cache, out, row_request, positions, block_tables)
     rows = q.shape[0]
-    _need(q.shape[1] == heads * key_dim and tuple(out.shape) == (rows, heads * value_dim) and q.dtype == out.dtype,
+    maps = (extras or NO_EXTRAS).maps
+    _need(q.shape[1] == heads * maps * key_dim and tuple(out.shape) == (rows, heads * value_dim) and q.dtype == out.dtype,
           "attention: q and out shapes do not fit")
-    _need(cache.dim() == 5 and cache.shape[1] == 1 and cache.shape[2] == kv_heads and cache.shape[4] == key_dim + value_dim,
+    _need(cache.dim() == 5 and cache.shape[1] == 1 and cache.shape[2] == kv_heads and cache.shape[4] == maps * key_dim + value_dim,
           "attention: cache layout does not fit")
     for t in (row_request, positions, block_tables):
         _need(t.dtype == torch.int32, "attention: metadata must be int32")
     _need(block_tables.dim() == 2 and row_request.numel() >= rows and positions.numel() >= rows, "attention: metadata shapes do not fit")
     splits = max(1, min(int(splits), 64))
-    partial = torch.empty((rows, heads, splits, value_dim + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
-    x = (extras or NO_EXTRAS).checked(heads, value_dim)
+    x = (extras or NO_EXTRAS).checked(heads, value_dim, rows)
+    partial = None
+    if splits > 1 or maps > 1 or staged:
+        partial = torch.empty((rows, heads * maps, splits, value_dim + 2), dtype=torch.float32, device=q.device)
+    heads = heads * maps                      # the kernels count map heads
     if staged:
-        if partial is None:
-            partial = torch.empty((rows, heads, 1, value_dim + 2), dtype=torch.float32, device=q.device)
         _check(_fn("attention_split", "llmx_attention_staged")(
             _ptr(q), _code(q), _ptr(cache), _code(cache), _ptr(out), _ptr(row_request), _ptr(positions), _ptr(block_tables),
             block_tables.shape[1], rows, heads, kv_heads, key_dim, value_dim, cache.shape[3], int(window or 0), int(chunk or 0),
@@ -821,22 +883,23 @@ def attention_split(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, row
     _check(_fn("attention_split", "llmx_attention_split")(
         _ptr(q), _code(q), _ptr(cache), _code(cache), _ptr(out), _ptr(row_request), _ptr(positions), _ptr(block_tables),
         block_tables.shape[1], rows, heads, kv_heads, key_dim, value_dim, cache.shape[3], int(window or 0), int(chunk or 0),
-        float(scale), splits, _ptr(partial), *x, _stream()), "attention_split", 2 if splits > 1 else 1)
+        float(scale), splits, _ptr(partial), *x, _stream()), "attention_split", 2 if splits > 1 or maps > 1 else 1)
     return out
 
 
-def attention_staged_fits(q_dtype: torch.dtype, cache_dtype: torch.dtype, heads: int, kv_heads: int, key_dim: int, value_dim: int) -> bool:
+def attention_staged_fits(q_dtype: torch.dtype, cache_dtype: torch.dtype, heads: int, kv_heads: int, key_dim: int, value_dim: int,
+                          maps: int = 1) -> bool:
     """Whether `attention_split(staged=True)` takes these types and sizes."""
     if q_dtype not in _CODE or cache_dtype not in _CODE:
         return False
     f = _fn("attention_split", "llmx_attention_staged_fits")
-    return bool(f(_CODE[q_dtype], _CODE[cache_dtype], int(heads), int(kv_heads), int(key_dim), int(value_dim)))
+    return bool(f(_CODE[q_dtype], _CODE[cache_dtype], int(heads) * int(maps), int(kv_heads), int(key_dim), int(value_dim), int(maps)))
 
 
-def attention_tiled_fits(heads: int, kv_heads: int, key_dim: int, value_dim: int) -> bool:
+def attention_tiled_fits(heads: int, kv_heads: int, key_dim: int, value_dim: int, maps: int = 1) -> bool:
     """Whether the tiled form of `attention_split` takes these sizes (it also wants bfloat16 queries and cache)."""
     f = _fn("attention_split", "llmx_attention_tiled_fits")
-    return bool(f(int(heads), int(kv_heads), int(key_dim), int(value_dim)))
+    return bool(f(int(heads) * int(maps), int(kv_heads), int(key_dim), int(value_dim), int(maps)))
 
 
 def attention_tiled(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, step, block_tables: torch.Tensor, heads: int,
@@ -848,14 +911,15 @@ def attention_tiled(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, ste
     _cuda(q, cache, out, block_tables)
     rows = q.shape[0]
     _need(q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16, "attention_tiled: bfloat16 queries, output and cache")
-    _need(q.shape[1] == heads * key_dim and tuple(out.shape) == (rows, heads * value_dim), "attention: q and out shapes do not fit")
-    _need(cache.dim() == 5 and cache.shape[1] == 1 and cache.shape[2] == kv_heads and cache.shape[4] == key_dim + value_dim,
+    maps = (extras or NO_EXTRAS).maps
+    _need(q.shape[1] == heads * maps * key_dim and tuple(out.shape) == (rows, heads * value_dim), "attention: q and out shapes do not fit")
+    _need(cache.dim() == 5 and cache.shape[1] == 1 and cache.shape[2] == kv_heads and cache.shape[4] == maps * key_dim + value_dim,
           "attention: cache layout does not fit")
     _need(block_tables.dtype == torch.int32 and block_tables.dim() == 2 and rows == step.rows, "attention: metadata does not fit")
     _check(_fn("attention_split", "llmx_attention_tiled")(
         _ptr(q), _ptr(cache), _ptr(out), _ptr(step.row_start), _ptr(step.row_count), _ptr(step.history), _ptr(block_tables),
-        block_tables.shape[1], rows, step.requests, heads, kv_heads, key_dim, value_dim, cache.shape[3], int(window or 0),
-        int(chunk or 0), float(scale), *(extras or NO_EXTRAS).checked(heads, value_dim), _stream()), "attention_tiled")
+        block_tables.shape[1], rows, step.requests, heads * maps, kv_heads, key_dim, value_dim, cache.shape[3], int(window or 0),
+        int(chunk or 0), float(scale), *(extras or NO_EXTRAS).checked(heads, value_dim, rows), _stream()), "attention_tiled")
     return out
 
 

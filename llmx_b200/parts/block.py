@@ -1,6 +1,7 @@
 """How a layer's parts are arranged.  PreNormBlock: x += mixer(norm(x)); x += ffn(norm(x)).
 ParallelBlock: x += mixer(norm(x)) + ffn(norm(x)), with one norm or one for each.  SandwichBlock: a norm before and after each sublayer and a factor
 on what enters the stream: x += m * norm_b(mixer(norm_a(x))); x += m * norm_d(ffn(norm_c(x))).
+PostNormBlock: a norm after each sublayer and none before: x += norm_a(mixer(x)); x += norm_b(ffn(x)).
 
 The names of the four parts (the prefixes of their tensors) are arguments, so
 the arrangement knows no architecture's tensor names.  When all four parts have a twin in the native runtime
@@ -237,3 +238,93 @@ class SandwichBlock(Part):
             h = self.pre_ffn_norm.forward(x, zero=flat[pad:])
             self.ffn.forward(h, step, out)
             self.post_ffn_norm.add_into(x, out, self.factor)
+
+
+class _Sublayer:
+    """What one sublayer of a `PostNormBlock` works in, for one step: `h`, the stream in the type its products read, and one
+    float32 buffer that holds its output and the outputs of its stored products.  Whoever writes the stream last makes `h`
+    and clears the first `cleared` floats of the buffer in the same launch (`RMSNorm.add_into(copy=, zero=)`)."""
+
+    def __init__(self, part: Part, x: torch.Tensor):
+        rows, width = x.shape
+        self.part, self.x, self.h = part, x, None
+        self.act = part.precision.act
+        final = getattr(part, "output_product", lambda: None)()
+        # The output is cleared when products add pieces into it (or when the part knows no other way than adding).
+        self.fresh = final is not None
+        n = rows * width
+        own = (n + 3) & ~3 if final is None or final.adds_pieces(rows) else 0
+        at, self.pieces = own, []
+        for lin in getattr(part, "stored_products", lambda: ())():
+            m = rows * lin.out_features
+            if lin.adds_pieces(rows) and m % 4 == 0:
+                self.pieces.append((lin, at, m))
+                at += m
+        self.flat = torch.empty(at, dtype=torch.float32, device=x.device) if at else None
+        self.out = self.flat[:n].view(rows, width) if own else torch.empty((rows, width), dtype=torch.float32, device=x.device)
+
+    def copy_target(self) -> Optional[torch.Tensor]:
+        """Where the stream's copy goes; on the 32-bit path the sublayer reads the stream itself."""
+        if self.act is torch.float32:
+            self.h = self.x
+            return None
+        self.h = torch.empty(self.x.shape, dtype=self.act, device=self.x.device)
+        return self.h
+
+    def hand_over(self) -> torch.Tensor:
+        """Gives the part its cleared outputs; returns the buffer it adds to (or stores in)."""
+        for lin, at, m in self.pieces:
+            self.part.cleared_outputs[id(lin)] = self.flat[at:at + m].view(self.x.shape[0], lin.out_features)
+        if self.fresh:
+            self.part.fresh_residual = True
+        return self.out
+
+
+class PostNormBlock(Part):
+    """x += mixer_norm(mixer(x)); then, with a feed-forward, x += ffn_norm(ffn(x)).  The sublayers read the stream as it is.
+
+    A sublayer's output lands in a buffer of its own; the norm after it adds into the stream, and the same launch makes what
+    comes next (the stream in the type its products read, the clearing of buffers that products add pieces into).  What
+    comes next may be the next block: the model names it in `step.extras["next_block"]`, and the block leaves it what it
+    made in `step.extras["handoff"]`.  A mixer with a bias on its output product (`defer_output_bias`) leaves it to the norm.
+    `ffn` and its norm may be None.  `names`: the prefixes of the four parts' tensors."""
+
+    def __init__(self, mixer: Part, mixer_norm: Part, ffn: Optional[Part], ffn_norm: Optional[Part], names=("mix", "norm1", "mlp", "norm2")):
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("post-norm block: a feed-forward comes with its norm")
+        self.mixer, self.mixer_norm, self.ffn, self.ffn_norm, self.names = mixer, mixer_norm, ffn, ffn_norm, tuple(names)
+        if hasattr(mixer, "defer_output_bias"):
+            mixer.defer_output_bias = True
+
+    def children(self) -> Dict[str, Part]:
+        return {n: p for n, p in zip(self.names, (self.mixer, self.mixer_norm, self.ffn, self.ffn_norm)) if p is not None}
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def forward(self, x: torch.Tensor, step: StepBatch, cache_entry, write_cache=True) -> None:
+        """x: the float32 residual stream [rows, hidden], updated in place."""
+        handed = step.extras.pop("handoff", None)
+        if handed is not None and handed[0] is self and handed[1].x is x:
+            mine = handed[1]
+        else:
+            mine = _Sublayer(self.mixer, x)
+            self.mixer_norm.add_into(x, None, copy=mine.copy_target(), zero=mine.flat)
+        following = step.extras.get("next_block")
+        following = following if isinstance(following, PostNormBlock) else None
+        after = _Sublayer(self.ffn, x) if self.ffn is not None else _Sublayer(following.mixer, x) if following else None
+        out = mine.hand_over()
+        self.mixer.forward(mine.h, step, cache_entry, out, write_cache)
+        bias = getattr(self.mixer, "output_bias", None) if getattr(self.mixer, "defer_output_bias", False) else None
+        self._join(self.mixer_norm, x, out, after, bias)
+        if self.ffn is not None:
+            mine, after = after, _Sublayer(following.mixer, x) if following else None
+            out = mine.hand_over()
+            self.ffn.forward(mine.h, step, out)
+            self._join(self.ffn_norm, x, out, after)
+        if after is not None:
+            step.extras["handoff"] = (following, after)
+
+    @staticmethod
+    def _join(norm: Part, x: torch.Tensor, out: torch.Tensor, after: Optional[_Sublayer], bias: Optional[torch.Tensor] = None) -> None:
+        norm.add_into(x, out, in_bias=bias, copy=None if after is None else after.copy_target(), zero=None if after is None else after.flat)

@@ -31,7 +31,7 @@ from .. import ops, runtime
 from ..cache.manager import KVSpec
 from ..weights.spec import TensorSpec
 from .base import Part, PartPlan, Precision, StepBatch, StepShape
-from .linear import Linear, stored_product
+from .linear import Linear, add_product, stored_product
 from .rope import blended_frequencies, power_frequencies
 
 
@@ -70,6 +70,9 @@ class LatentAttention(Part):
     def stored_products(self):
         """The products whose result is stored (not added to the residual): a block may clear their outputs in passing."""
         return (self.down, self.uq) if self.q_rank else (self.down,)
+
+    def output_product(self) -> Linear:
+        return self.o
 
     def cache_spec(self):
         return KVSpec(1, self.kv_rank + self.rot_dim, self.window, planes=1)
@@ -175,4 +178,4 @@ class LatentAttention(Part):
                                  self.scale, halves=halves, magnitude=mag)
         if self.gate:
             ops.sigmoid_gate_(o, proj[:, gate_at:gate_at + self.v_width])
-        self.o(o, out=residual, accumulate=True)
+        add_product(self, self.o, o, residual)

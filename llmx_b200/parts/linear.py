@@ -52,6 +52,17 @@ def stored_product(part, lin: "Linear", a: torch.Tensor) -> torch.Tensor:
     return lin(a)
 
 
+def add_product(part, lin: "Linear", a: torch.Tensor, residual: torch.Tensor) -> None:
+    """residual += lin(a), the last product of a sublayer.  A block whose `residual` is a buffer of this sublayer's own says so
+    with `part.fresh_residual` (True for the one call): the product is then stored.  (The block cleared the buffer if the
+    product adds pieces, and left it as it was otherwise.)"""
+    if getattr(part, "fresh_residual", False):
+        part.fresh_residual = False
+        lin(a, out=residual, cleared=lin.adds_pieces(a.shape[0]))
+    else:
+        lin(a, out=residual, accumulate=True)
+
+
 class Linear:
     def __init__(self, weight: torch.Tensor, precision: Precision):
         # A weight stored in 32-bit is rounded once for the bfloat16 path; a bfloat16 weight

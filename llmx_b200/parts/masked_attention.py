@@ -39,6 +39,13 @@ Options for designs that vary it (any of them makes the rows go through the gene
                           no key and no value; "zero": a sink of 0 (one is added to the denominator)
     rotate_values True    the value of position j is rotated by j over all of V (pair m by j * rot_base^(-2m / V), no scaling,
                           in the q/k pairing) and cached so; a row's output is turned back by its own position
+    difference d          differential attention: every query and key head is two maps of D values ([map 1, map 2], normed and
+                          rotated each by itself) over the same values; with a1, a2 their attentions and the layer's number
+                          lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + d (four vectors of D under `difference_roles`), the head's
+                          output is o = a1 - lambda a2, o / sqrt(mean(o^2) + difference_eps) * (1 - d).  A cache row is
+                          [key 1 ; key 2 ; value]; both maps, the difference and its norm are one kernel (or the merge of one)
+    head_gate True        head h's output times sigmoid(h Wg^T)_h, one number a head (role `gate_role`; its rows join the stacked
+                          product), in the kernel that makes the output
 With a filter the mixer's cache need is a pair (keys and values, filter state) and `forward` is handed a pair of entries.
 
     rounded_weights True  the design lets softmax weights enter the product with the values rounded to bfloat16 (the
@@ -61,7 +68,7 @@ from .. import ops, runtime
 from ..cache.manager import KVSpec, StateSpec
 from ..weights.spec import TensorSpec
 from .base import Part, Precision, StepBatch
-from .linear import Linear, stored_product
+from .linear import Linear, add_product, stored_product
 
 
 class MaskedAttention(Part):
@@ -71,7 +78,8 @@ class MaskedAttention(Part):
                  names=("q", "k", "v", "o", "q.norm", "k.norm"), bias: bool = False, taps: int = 1, pairing: str = "halves",
                  qk_norm: str = "before", qk_norm_weight: bool = True, shared_kv: bool = False, rounded_weights: bool = False,
                  output_bias: Optional[bool] = None, rot_freq=None, rot_magnitude: float = 1.0, softcap: Optional[float] = None,
-                 sink: Optional[str] = None, rotate_values: bool = False, sink_role: str = "sink"):
+                 sink: Optional[str] = None, rotate_values: bool = False, sink_role: str = "sink", difference: Optional[float] = None,
+                 difference_eps: float = 0.0, difference_roles=("lq1", "lk1", "lq2", "lk2"), head_gate: bool = False, gate_role: str = "g"):
         if heads % kv_heads:
             raise ValueError("attention: head count must be divisible by the key/value head count")
         if rot_dims % 2 or rot_dims > key_dim or rot_dims < 0:
@@ -82,12 +90,18 @@ class MaskedAttention(Part):
         self.qk_norm_eps = qk_norm_eps
         self.rot_dims, self.rot_base, self.rot_factor = int(rot_dims), float(rot_base), float(rot_factor)
         self.window, self.chunk, self.names = window, chunk, tuple(names)
-        self.q_width, self.k_width, self.v_width = self.heads * self.key_dim, self.kv_heads * self.key_dim, self.kv_heads * self.value_dim
+        self.difference, self.difference_eps = None if difference is None else float(difference), float(difference_eps)
+        self.difference_roles, self.head_gate, self.gate_role = tuple(difference_roles), bool(head_gate), gate_role
+        self.maps = 1 if difference is None else 2
+        self.q_width, self.k_width = self.heads * self.maps * self.key_dim, self.kv_heads * self.maps * self.key_dim
+        self.v_width = self.kv_heads * self.value_dim
         self.o_width = self.heads * self.value_dim
         if pairing not in ("halves", "neighbours") or qk_norm not in ("before", "after", "whole") or taps < 1:
             raise ValueError("attention: pairing is halves or neighbours, qk_norm before, after or whole, the filter has at least one tap")
         if sink not in (None, "learned", "zero") or (softcap is not None and not softcap > 0):
             raise ValueError("attention: sink is learned, zero or None; a cap on the scores is positive")
+        if difference is not None and (sink is not None or rotate_values):
+            raise ValueError("attention: two maps come without a sink and without rotated values")
         if rotate_values and self.value_dim % 2:
             raise ValueError("attention: rotated values need an even value width")
         if rot_freq is not None and len(rot_freq) != rot_dims // 2:
@@ -99,8 +113,8 @@ class MaskedAttention(Part):
         self.bias, self.taps, self.pairing, self.qk_norm = bool(bias), int(taps), pairing, qk_norm
         self.qk_norm_weight, self.shared_kv = bool(qk_norm_weight), bool(shared_kv)
         self.general = (self.bias or self.taps > 1 or pairing != "halves" or qk_norm != "before" or not self.qk_norm_weight or self.shared_kv
-                        or self.rot_magnitude != 1.0 or self.rotate_values)
-        plain_softmax = softcap is None and sink is None and not self.rotate_values
+                        or self.rot_magnitude != 1.0 or self.rotate_values or self.maps > 1 or self.head_gate)
+        plain_softmax = softcap is None and sink is None and not self.rotate_values and self.maps == 1 and not self.head_gate
         self.channels = self.q_width + (0 if self.shared_kv else self.k_width + self.v_width)
         # Whether the paged kernels can serve this geometry (decided for good in `load`, which knows the path's type).
         self.paged_shape = None
@@ -117,8 +131,12 @@ class MaskedAttention(Part):
     def children(self):
         return {"paged": self.paged_shape} if self.paged_shape is not None else {}
 
+    def output_product(self) -> Linear:
+        return self.o
+
     def cache_spec(self):
-        kv = KVSpec(self.kv_heads, self.key_dim, self.window) if self.paged else KVSpec(self.kv_heads, self.key_dim + self.value_dim, self.window, planes=1, chunk=self.chunk)
+        kv = KVSpec(self.kv_heads, self.key_dim, self.window) if self.paged else KVSpec(self.kv_heads, self.maps * self.key_dim + self.value_dim, self.window,
+                                                                                                       planes=1, chunk=self.chunk)
         if self.taps > 1:
             return (kv, StateSpec(((self.taps - 1) * self.channels,), "float32"))
         return kv
@@ -140,6 +158,11 @@ class MaskedAttention(Part):
             specs[qn] = TensorSpec((self.q_width if whole else self.key_dim,), "vector", init="one_plus_normal", std=0.01)
             if not self.shared_kv:
                 specs[kn] = TensorSpec((self.k_width if whole else self.key_dim,), "vector", init="one_plus_normal", std=0.01)
+        if self.difference is not None:
+            for name in self.difference_roles:
+                specs[name] = TensorSpec((self.key_dim,), "vector", init="normal", std=0.1)
+        if self.head_gate:
+            specs[self.gate_role] = TensorSpec((self.heads, self.hidden))
         if self.sink == "learned":
             specs[self.sink_role] = TensorSpec((self.heads,), "vector", init="normal", std=1.0)
         return specs
@@ -157,7 +180,8 @@ class MaskedAttention(Part):
         self._staged = {}                    # by the cache's type: whether the staged form of the plain attention takes these sizes
         q, k, v, o, qn, kn = self.names
         made = [q] if self.shared_kv else [q, k, v]
-        self.qkv = Linear(torch.cat([tensors[n] for n in made], dim=0), precision)
+        stacked = made + ([self.gate_role] if self.head_gate else [])
+        self.qkv = Linear(torch.cat([tensors[n] for n in stacked], dim=0), precision)
         self.o = Linear(tensors[o], precision)
         self.q_norm = self.k_norm = None
         if self.qk_norm_eps is not None and self.qk_norm_weight:
@@ -172,13 +196,19 @@ class MaskedAttention(Part):
             self.vfreq = torch.from_numpy(np.power(np.float64(self.rot_base), -2.0 * m / self.value_dim).astype(np.float32)).to(dev)
         sink = tensors[self.sink_role].to(torch.float32).contiguous() if self.sink == "learned" else self.sink
         self.extras = None
-        if self.softcap is not None or self.sink is not None or self.rotate_values:
-            self.extras = ops.SoftmaxExtras(self.softcap, sink, self.vfreq, self.pairing == "neighbours")
+        difference = None
+        if self.difference is not None:
+            # One number a layer, made once in double precision.
+            a, b, c, d = (tensors[n].to(device="cpu", dtype=torch.float64) for n in self.difference_roles)
+            self.difference_factor = float(torch.exp(torch.dot(a, b)) - torch.exp(torch.dot(c, d))) + self.difference
+            difference = (self.difference_factor, 1.0 - self.difference, self.difference_eps)
+        if self.softcap is not None or self.sink is not None or self.rotate_values or difference is not None or self.head_gate:
+            self.extras = ops.SoftmaxExtras(self.softcap, sink, self.vfreq, self.pairing == "neighbours", difference)
         self.taps_w = torch.cat([tensors[n + ".conv"] for n in made], dim=0).to(torch.float32).contiguous() if self.taps > 1 else None
         self.freq = torch.from_numpy(self.frequencies()).to(self.o.weight.device) if self.rot_dims else None
         self.paged = self.paged_shape is not None and precision.act is torch.bfloat16 and not precision.invariant
         self.tiled = precision.act is torch.bfloat16 and not precision.invariant and \
-            ops.attention_tiled_fits(self.heads, self.kv_heads, self.key_dim, self.value_dim)
+            ops.attention_tiled_fits(self.heads, self.kv_heads, self.key_dim, self.value_dim, self.maps)
 
     def forward(self, h: torch.Tensor, step: StepBatch, cache_entry, residual: torch.Tensor, write_cache=True) -> None:
         """`cache_entry`: the entry of keys and values, or with a filter the pair (keys and values, filter state);
@@ -194,7 +224,11 @@ class MaskedAttention(Part):
                 and residual.dtype is torch.float32 and residual.is_contiguous() and tuple(residual.shape) == (rows, self.hidden)):
             raise runtime.KernelError("attention: rows of the path's type and the mixer's width, a float32 residual")
         group, cache = step.kv(cache_entry)
-        proj = stored_product(self, self.qkv, h)                             # [rows, q | k | v], 32-bit
+        proj = stored_product(self, self.qkv, h)                             # [rows, q | k | v (| gate)], 32-bit
+        extras = self.extras
+        if self.head_gate:
+            proj, gate = proj[:, :self.channels], proj[:, self.channels:]
+            extras = extras.with_gate(gate)
         q = torch.empty((rows, self.q_width), dtype=self.precision.act, device=h.device)
         slots = group.slots if write_cache else torch.full_like(group.slots, -1)
         if self.general or self.paged:
@@ -203,7 +237,7 @@ class MaskedAttention(Part):
                            taps_w=self.taps_w, state=step.state(state_entry) if self.taps > 1 else None,
                            norm="none" if self.qk_norm_eps is None else self.qk_norm, q_weight=self.q_norm, k_weight=self.k_norm,
                            eps=float(self.qk_norm_eps or 0.0), freq=self.freq, neighbours=self.pairing == "neighbours",
-                           rot_mag=self.rot_magnitude, vfreq=self.vfreq)
+                           rot_mag=self.rot_magnitude, vfreq=self.vfreq, maps=self.maps)
         else:
             ops.qk_norm_rope_write(proj, self.heads, self.kv_heads, self.key_dim, self.value_dim, self.q_norm, self.k_norm,
                                    float(self.qk_norm_eps or 0.0), self.freq, step.positions, slots, q, cache)
@@ -216,21 +250,21 @@ class MaskedAttention(Part):
             ops_attn.paged_attention(q, o, step, cache_entry, self.heads, self.kv_heads, self.key_dim, self.window, self.scale)
         elif self.tiled and step.max_row_count > 4 and cache.dtype is torch.bfloat16:
             ops.attention_tiled(q, cache, o, step, group.block_tables, self.heads, self.kv_heads, self.key_dim, self.value_dim,
-                                self.window, self.chunk, self.scale, extras=self.extras)
+                                self.window, self.chunk, self.scale, extras=extras)
         else:
             span = min(x for x in (step.max_context, self.window, self.chunk) if x)
             staged = self._staged.get(cache.dtype)
             if staged is None:
                 staged = self._staged[cache.dtype] = not self.precision.invariant and ops.attention_staged_fits(
-                    q.dtype, cache.dtype, self.heads, self.kv_heads, self.key_dim, self.value_dim)
+                    q.dtype, cache.dtype, self.heads, self.kv_heads, self.key_dim, self.value_dim, self.maps)
             if staged:
                 # A block a (row, key/value head, range of keys): enough ranges to fill the device three blocks an SM.
                 splits = max(1, min(64, span // 128, 444 // max(rows * self.kv_heads, 1)))
             else:
-                splits = 1 if self.precision.invariant else max(1, min(32, span // 128, 2368 // max(rows * self.heads, 1)))
+                splits = 1 if self.precision.invariant else max(1, min(32, span // 128, 2368 // max(rows * self.heads * self.maps, 1)))
             ops.attention_split(q, cache, o, step.row_request, step.positions, group.block_tables, self.heads, self.kv_heads,
-                                self.key_dim, self.value_dim, self.window, self.chunk, self.scale, splits=splits, extras=self.extras,
+                                self.key_dim, self.value_dim, self.window, self.chunk, self.scale, splits=splits, extras=extras,
                                 staged=staged)
-        self.o(o, out=residual, accumulate=True)
+        add_product(self, self.o, o, residual)
         if self.output_bias is not None and not self.defer_output_bias:
             ops.add_bias_(residual, self.output_bias)

@@ -14,7 +14,7 @@ import torch
 from .. import runtime
 from ..weights.spec import TensorSpec
 from .base import NativeHandle, Part, Precision, StepBatch
-from .linear import ActivatedLinear, Linear, call_struct
+from .linear import ActivatedLinear, Linear, add_product, call_struct
 
 
 class GatedMLP(Part):
@@ -86,6 +86,9 @@ class ClampedGLU(Part):
     def stored_products(self):
         return (self.gate_up,)
 
+    def output_product(self) -> Linear:
+        return self.down
+
     def load(self, tensors, precision: Precision) -> None:
         super().load(tensors, precision)
         self.cleared_outputs = {}
@@ -98,7 +101,7 @@ class ClampedGLU(Part):
         if not (h.is_cuda and h.is_contiguous() and h.dtype is self.precision.act and tuple(h.shape) == (rows, self.hidden)
                 and residual.dtype is torch.float32 and residual.is_contiguous() and tuple(residual.shape) == (rows, self.hidden)):
             raise runtime.KernelError("feed-forward: rows of the path's type and the part's width, a float32 residual")
-        self.down(self.gate_up.activated(self, h), out=residual, accumulate=True)
+        add_product(self, self.down, self.gate_up.activated(self, h), residual)
 
 
 class ActivatedMLP(Part):

@@ -77,6 +77,19 @@ class RMSNorm(Part):
         ops.rmsnorm_pair(x, self.weight, other.weight, self.eps, both[0], both[1], zero=zero)
         return both[0], both[1]
 
+    def add_into(self, residual: torch.Tensor, y: Optional[torch.Tensor], factor: float = 1.0, in_bias: Optional[torch.Tensor] = None,
+                 copy: Optional[torch.Tensor] = None, zero: Optional[torch.Tensor] = None) -> None:
+        """residual += norm(y + in_bias), float32 rows (the norm after a sublayer); `copy` takes the new residual in its own type and
+        `zero`, a float32 buffer, is cleared, all in one launch.  Without y: copy and clearing alone."""
+        from .. import ops
+        if factor != 1.0:
+            raise runtime.KernelError("rmsnorm: the kernel that adds the normed rows has no factor")
+        if zero is not None and (zero.numel() % 4 or zero.data_ptr() % 16):
+            zero.zero_()
+            zero = None
+        if y is not None or copy is not None or zero is not None:
+            ops.rmsnorm_add_(residual, y, self.weight, self.eps, in_bias=in_bias, copy=copy, zero=zero)
+
     def pairs_with(self, other: Part) -> bool:
         return type(other) is RMSNorm and other.width == self.width and other.eps == self.eps
 

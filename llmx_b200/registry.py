@@ -96,3 +96,4 @@ def _ensure_builtin() -> None:
     from .models import zamizen as _zamizen  # noqa: F401
     from .models import nomutar as _nomutar  # noqa: F401
     from .models import fipadra as _fipadra  # noqa: F401
+    from .models import dikusun as _dikusun  # noqa: F401
