@@ -140,6 +140,10 @@ def reference_arm(args):
 # second layer's feed-forward Kisepel's experts with 4 identity experts beside them, in 5 groups of which 3 are kept, the others'
 # dense) beside the two models that have its kernels' nearest relatives: the Buzetar (the same three kinds of mixers) and the
 # Nomutar (routed experts under a gated shared unit).
+# `--design dikusun`: a Dikusun of as many layers (latent attention, differential attention under the window with heads of two maps
+# of 64 over values of 128, gated linear attention in turn; every feed-forward Buzetar's) beside the three models that have its
+# kernels' nearest relatives: the Buzetar (latent attention, the delta rule, the same feed-forward), the Nomutar (capped
+# attention under a window) and the Kisepel (a recurrence with a decay per key channel).
 DESIGN_SIZES = {
     "w2048": dict(width=2048, heads=16, ff=6144, vocab=32768, q_rank=768, kv_rank=512, rot=64, window=2048, layers=6),
     "w4096": dict(width=4096, heads=32, ff=12288, vocab=32768, q_rank=1536, kv_rank=512, rot=64, window=4096, layers=3),
@@ -153,7 +157,7 @@ def design_bench(args) -> int:
     import statistics
     import torch
     from llmx_b200 import ops
-    from llmx_b200.config import BuzetarConfig, FipadraConfig, KisepelConfig, NomutarConfig, Qwen3Config, ZamizenConfig
+    from llmx_b200.config import BuzetarConfig, DikusunConfig, FipadraConfig, KisepelConfig, NomutarConfig, Qwen3Config, ZamizenConfig
     from llmx_b200.engine import Engine, EngineOptions, StepEntry
     from llmx_b200.engine.decode_loop import DecodeSession
     torch.cuda.set_device(0)
@@ -221,7 +225,7 @@ def design_bench(args) -> int:
             buz_latent = BuzetarConfig.from_dict({"architecture": "Buzetar", "vocab": z["vocab"], "width": E, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
                                                   "logit_scale": 1.0, "layers": [all_latent] * L})
             runs = (("zamizen", zam), ("buzetar_latent", buz_latent), ("qwen3", qwen))
-        if args.design in ("nomutar", "fipadra"):
+        if args.design in ("nomutar", "fipadra", "dikusun"):
             G = max(H // 4, 1)
             head = {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
             ramp = {"base": 1000000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 16.0, "slow": 2.0}}
@@ -249,6 +253,15 @@ def design_bench(args) -> int:
             fip = FipadraConfig.from_dict({"architecture": "Fipadra", "vocab": z["vocab"], "width": E, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
                                            "layers": [dict(fip_mixers[i % 3], mlp=fip_mlps[i % 2]) for i in range(L)]})
             runs = (("fipadra", fip), ("buzetar", buz), ("nomutar", nom))
+        if args.design == "dikusun":
+            dik_mixers = [
+                {"type": "latent_attention", "mixer": {"heads": H, "dim": 128, "vdim": 128, "q_rank": z["q_rank"], "kv_rank": z["kv_rank"], "scale": 128 ** -0.5}},
+                {"type": "attention", "mixer": {"heads": H, "kv_heads": max(H // 4, 1), "dim": 64, "vdim": 128, "scale": 0.125, "softcap": 40.0, "diff": 0.4,
+                                                "mask": {"size": z["window"]}, "rot": {"base": 1000000.0, "dims": 64}}},
+                {"type": "gla", "mixer": {"heads": H, "dim": 128, "vdim": 128, "tau": 12.0, "decay_rank": 32}}]
+            dik = DikusunConfig.from_dict({"architecture": "Dikusun", "vocab": z["vocab"], "width": E, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0},
+                                           "layers": [dict(dik_mixers[i % 3], mlp=mlp) for i in range(L)]})
+            runs = (("dikusun", dik), ("buzetar", buz), ("nomutar", nom), ("kisepel", kis))
         res = {"config": dict(z)}
         out["sizes"][name] = res                                # filled as the arms end, so that a run that stops early says what it has
         for tag, cfg in runs:
@@ -331,11 +344,11 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true")
     ap.add_argument("--only", choices=["decode", "prefill", "sample"], default=None,
                     help="run one part only (for profiling); the line then holds only that part")
-    ap.add_argument("--design", choices=["buzetar", "kisepel", "zamizen", "nomutar", "fipadra"], default=None,
+    ap.add_argument("--design", choices=["buzetar", "kisepel", "zamizen", "nomutar", "fipadra", "dikusun"], default=None,
                     help="instead of the default workload: prompt and decode throughput of this design at sizes that resemble a "
                          "real model's layers, beside the closest other design of equal size (Buzetar beside Qwen3, Kisepel beside Buzetar, "
-                         "Zamizen beside an all-latent Buzetar and Qwen3, Nomutar beside an all-attention Zamizen and Kisepel, Fipadra beside Buzetar "
-                         "and Nomutar; one JSON line of its own)")
+                         "Zamizen beside an all-latent Buzetar and Qwen3, Nomutar beside an all-attention Zamizen and Kisepel, Fipadra beside Buzetar and Nomutar, "
+                         "Dikusun beside Buzetar, Nomutar and Kisepel; one JSON line of its own)")
     ap.add_argument("--design-size", default=None, help="with --design: one of " + ", ".join(sorted(DESIGN_SIZES)) + " (default: all)")
     args = ap.parse_args()
     if args.impl == "reference":

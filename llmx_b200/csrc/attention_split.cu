@@ -535,7 +535,8 @@ static int launch_merge(const float* partial, void* out, int q_dtype, int rows, 
 // buffers of shared memory by cp.async (16-byte pieces, the next tile in flight while this one is used; rows padded by
 // one piece, so that lanes reading 16-byte pieces of 32 different rows meet in no bank).  Warp w serves heads w, w + 4, ...:
 // a lane makes the whole score of one key (no shuffles within a key), the tile's maximum and sum meet once a tile, the
-// 32-bit weights lie in shared memory and every lane adds them over its columns of the values.  Every (row, head, range)
+// 32-bit weights lie in shared memory and every lane adds them over its pairs of columns of the values, read once for the
+// warp's heads.  Every (row, head, range)
 // leaves sum, maximum and weight in `partial`, which the merge kernel above finishes (sink, division, turning back).
 template <typename T> struct Piece;
 template <> struct Piece<float> {
@@ -557,6 +558,9 @@ template <> struct Piece<__nv_bfloat16> {
         }
     }
 };
+
+__device__ __forceinline__ float2 read_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 read_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 
 template <typename T, int HPW, int VPL>
 __global__ void __launch_bounds__(128)
@@ -654,18 +658,34 @@ attention_staged_kernel(const T* __restrict__ q, const T* __restrict__ cache, co
             l[hh] = l[hh] * corr + lsum;                 // per lane; the lanes meet at the end
 #pragma unroll
             for (int i = 0; i < VPL; ++i) acc[hh][i] *= corr;
-            __syncwarp();
-            for (int key = 0; key < n_here; ++key) {
-                const float e = ph[key];
-                const T* vr = buf + (size_t)key * ws + maps * D;
+        }
+        __syncwarp();
+        // The values once for all of the warp's heads, four keys at a time (past the last key weights and values are zeros).
+        if (warp < ratio) {
+            for (int key = 0; key < n_here; key += 4) {
+                float4 e[HPW];
 #pragma unroll
-                for (int i = 0; i < VPL; ++i) {
-                    const int c = lane + 32 * i;
-                    if (c < V) acc[hh][i] = fmaf(e, to_float(vr[c]), acc[hh][i]);
+                for (int hh = 0; hh < HPW; ++hh)
+                    e[hh] = warp + 4 * hh < ratio ? *reinterpret_cast<const float4*>(ps + (size_t)(warp + 4 * hh) * TK + key) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const T* vr = buf + (size_t)(key + j) * ws + maps * D;
+#pragma unroll
+                    for (int i = 0; i < VPL; i += 2) {
+                        const int c = 2 * lane + 32 * i;
+                        if (c >= V) continue;
+                        const float2 v = read_pair(vr + c);
+#pragma unroll
+                        for (int hh = 0; hh < HPW; ++hh) {
+                            const float w = j == 0 ? e[hh].x : j == 1 ? e[hh].y : j == 2 ? e[hh].z : e[hh].w;
+                            acc[hh][i] = fmaf(w, v.x, acc[hh][i]);
+                            acc[hh][i + 1] = fmaf(w, v.y, acc[hh][i + 1]);
+                        }
+                    }
                 }
             }
-            __syncwarp();                                // the weights are written again at the next tile
         }
+        __syncwarp();                                    // the weights are written again at the next tile
     }
 #pragma unroll
     for (int hh = 0; hh < HPW; ++hh) {
@@ -674,9 +694,9 @@ attention_staged_kernel(const T* __restrict__ q, const T* __restrict__ cache, co
         const float lt = warp_sum(l[hh]);
         float* prow = partial + (((size_t)row * heads + (size_t)g * ratio + hl) * splits + split) * (size_t)(V + 2);
 #pragma unroll
-        for (int i = 0; i < VPL; ++i) {
-            const int c = lane + 32 * i;
-            if (c < V) prow[c] = acc[hh][i];
+        for (int i = 0; i < VPL; i += 2) {
+            const int c = 2 * lane + 32 * i;
+            if (c < V) prow[c] = acc[hh][i], prow[c + 1] = acc[hh][i + 1];
         }
         if (lane == 0) {
             prow[V] = m[hh];

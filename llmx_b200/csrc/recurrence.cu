@@ -30,6 +30,7 @@
 // [heads * D]).
 #include "common.cuh"
 #include <math.h>
+#include <type_traits>
 
 namespace {
 constexpr int REC_THREADS = 128;
@@ -150,10 +151,14 @@ recurrence_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     }
 }
 
-// The wide form for long runs of rows: a warp a column, eight columns of one head a block, and the rows' q, k, v and
-// gates brought to shared memory sixteen rows at a time by cp.async (the next sixteen in flight meanwhile), so that
-// a row waits for shared memory and for the row before it, not for the L2 cache.
-constexpr int WIDE_THREADS = 256, WIDE_COLS = 8, WIDE_CH = 16;
+// The wide form for long runs of rows: sixteen columns of one head a block, and the rows' q, k, v and gates brought to shared
+// memory sixteen rows at a time by cp.async (the next sixteen in flight meanwhile), so that a row waits for shared memory
+// and for the row before it, not for the L2 cache.  With a delta rule a warp owns one column: every row waits for a sum over
+// the warp's lanes.  Without one a warp owns two columns (a row's q, k and gates are read once for both) and the
+// read-outs of eight rows are summed over the lanes together.
+constexpr int WIDE_COLS = 16, WIDE_CH = 16, WIDE_SUMS = 8;
+constexpr int wide_columns_a_warp(int mode) { return mode == M_DELTA || mode == M_DELTA_VEC ? 1 : 2; }
+constexpr int wide_threads(int mode) { return 32 * WIDE_COLS / wide_columns_a_warp(mode); }
 
 __device__ __forceinline__ void cp_async_4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -163,24 +168,27 @@ __device__ __forceinline__ void cp_async_16f(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// A lane holds the PER neighbouring values d = PER * lane .. of its column, so that a row's q and k are one
-// 16-byte read each from shared memory when PER is 4.
+// A lane holds the PER neighbouring values d = PER * lane .. of its column; a row's vectors are padded with zeros to PER * 32
+// values, so that a lane's share is whole 16-byte (or 8-byte) reads from shared memory without a condition.
 template <int PER>
-__device__ __forceinline__ void read_run(const float* p, int lane, int D, float (&out)[PER]) {
-    if (PER == 4 && D % 4 == 0) {
-        const float4 x = lane * 4 < D ? *reinterpret_cast<const float4*>(p + lane * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-        out[0] = x.x;
-        out[1] = x.y;
-        out[2] = x.z;
-        out[3] = x.w;
+__device__ __forceinline__ void read_run(const float* p, int lane, float (&out)[PER]) {
+    static_assert(PER == 1 || PER == 2 || PER % 4 == 0, "a lane's share of a row");
+    if constexpr (PER == 1) {
+        out[0] = p[lane];
+    } else if constexpr (PER == 2) {
+        const float2 x = *reinterpret_cast<const float2*>(p + lane * 2);
+        out[0] = x.x, out[1] = x.y;
     } else {
 #pragma unroll
-        for (int i = 0; i < PER; ++i) out[i] = lane * PER + i < D ? p[lane * PER + i] : 0.0f;
+        for (int i = 0; i < PER; i += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(p + lane * PER + i);
+            out[i] = x.x, out[i + 1] = x.y, out[i + 2] = x.z, out[i + 3] = x.w;
+        }
     }
 }
 
 template <int PER, int MODE>
-__global__ void __launch_bounds__(WIDE_THREADS)
+__global__ void __launch_bounds__(wide_threads(MODE))
 recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, int q_stride,
                        int k_stride, int v_stride, const float* __restrict__ decay, const float* __restrict__ gate,
                        const float* __restrict__ beta, int gate_stride, int beta_stride, const float* __restrict__ skip,
@@ -190,53 +198,54 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
                        const int* __restrict__ slot_out, float* __restrict__ out, int heads, int qk_heads, int D, int V) {
     pdl_trigger();
     pdl_wait();
-    extern __shared__ __align__(16) float stage[];   // [2][WIDE_CH][row_floats]: q (Dp), k (Dp), [gates per channel (Dp)], v (8 columns), gate, beta, pad
+    extern __shared__ __align__(16) float stage[];   // [2][WIDE_CH][row_floats]: q (Dp), k (Dp), [gates per channel (Dp)], v (the block's columns), gate, beta, pad
     constexpr bool VEC = has_channel_gate(MODE);
+    constexpr int CPW = wide_columns_a_warp(MODE), THREADS = wide_threads(MODE);
     constexpr int NV = VEC ? 3 : 2;                  // vectors of D values a row brings
-    const int Dp = PER * 32;                         // a row's q and k padded to the lanes' runs (the pad is never written: zeros are read by the guard)
+    const int Dp = PER * 32;                         // a row's q and k padded to the lanes' runs (the pad is cleared once and never written by the copies)
     const int row_floats = NV * Dp + WIDE_COLS + 4;  // a multiple of 4: every row starts on 16 bytes
     const int r = blockIdx.x;
     const int blocks_per_head = (V + WIDE_COLS - 1) / WIDE_COLS;
     const int h = blockIdx.y / blocks_per_head;
     const int first_col = (blockIdx.y % blocks_per_head) * WIDE_COLS;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int col = first_col + warp;
+    const int col = first_col + warp * CPW;          // the warp's first column; columns past V shadow the last one and store nothing
     const int n = row_count[r];
     if (n <= 0) return;
-    const bool live = col < V;
-    const int j = live ? col : V - 1;
     const int a0 = row_start[r];
     const int hq = h / (heads / qk_heads);
-    float S[PER];
-    const float* sin_ = state + (size_t)slot_in[r] * slot_floats + ((size_t)h * V + j) * D;
+    float S[CPW][PER];
     const bool fresh = history[r] == 0;
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        const int d = lane * PER + i;
-        S[i] = (!fresh && d < D) ? sin_[d] : 0.0f;
+    for (int w = 0; w < CPW; ++w) {
+        const float* sin_ = state + (size_t)slot_in[r] * slot_floats + ((size_t)h * V + min(col + w, V - 1)) * D;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int d = lane * PER + i;
+            S[w][i] = (!fresh && d < D) ? sin_[d] : 0.0f;
+        }
     }
     const float dec = MODE == M_CONST ? decay[h] : VEC ? 1.0f : 0.0f;
     const float sk = MODE == M_SCALED && skip != nullptr ? skip[h] : 0.0f;
     // What this thread copies of every chunk is the same from chunk to chunk, so its places are worked out once:
-    // pieces of 16 bytes of q and k when rows allow it (else single values), and one of the chunk's small values.
+    // pieces of 16 bytes of q and k when rows allow it (else single values), and the chunk's small values one by one.
     const bool vec = D % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 &&
                      (!VEC || (gate_stride % 4 == 0 && ((uintptr_t)gate & 15) == 0));
     const int unit = vec ? 4 : 1;
     const int per_vec = D / unit;
     const int per_row = NV * per_vec;                // copies a row's q and k (and channel gates) take
-    constexpr int MAX_COPIES = NV * PER * 32 * WIDE_CH / WIDE_THREADS;     // at most, with single values
-    const int small_t = threadIdx.x / (WIDE_COLS + 2), small_e = threadIdx.x % (WIDE_COLS + 2);
+    constexpr int MAX_COPIES = NV * PER * 32 * WIDE_CH / THREADS;     // at most, with single values
     auto issue = [&](int chunk, int which) {
         float* buf = stage + (size_t)which * WIDE_CH * row_floats;
         const int t0 = chunk * WIDE_CH, rows = min(WIDE_CH, n - t0);
         const int copies = rows * per_row;
         int p = threadIdx.x, t = p / per_row, e = p % per_row;
-        const int dt = WIDE_THREADS / per_row, de = WIDE_THREADS % per_row;
+        const int dt = THREADS / per_row, de = THREADS % per_row;
 #pragma unroll 4
         for (int i = 0; i < MAX_COPIES; ++i) {
             if (p >= copies) break;
             const size_t row = (size_t)(a0 + t0 + t);
-            const int which_vec = e / per_vec;       // 0: q, 1: k, 2: the gates per channel
+            const int which_vec = (e >= per_vec) + (e >= 2 * per_vec);       // 0: q, 1: k, 2: the gates per channel
             const int off = (e - which_vec * per_vec) * unit;
             const float* src = which_vec == 0 ? q + row * q_stride + (size_t)hq * D + off
                              : which_vec == 1 ? k + row * k_stride + (size_t)hq * D + off
@@ -244,7 +253,7 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
             float* dst = buf + (size_t)t * row_floats + which_vec * Dp + off;
             if (vec) cp_async_16f(dst, src);
             else cp_async_4(dst, src);
-            p += WIDE_THREADS;
+            p += THREADS;
             t += dt;
             e += de;
             if (e >= per_row) {
@@ -252,7 +261,9 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
                 ++t;
             }
         }
-        if (small_t < rows && (small_e < WIDE_COLS || (small_e == WIDE_COLS ? (MODE == M_DELTA || MODE == M_SCALED) : has_beta(MODE)))) {
+        for (int i = threadIdx.x; i < WIDE_CH * (WIDE_COLS + 2); i += THREADS) {
+            const int small_t = i / (WIDE_COLS + 2), small_e = i % (WIDE_COLS + 2);
+            if (small_t >= rows || !(small_e < WIDE_COLS || (small_e == WIDE_COLS ? (MODE == M_DELTA || MODE == M_SCALED) : has_beta(MODE)))) continue;
             const size_t row = (size_t)(a0 + t0 + small_t);
             const float* src = small_e < WIDE_COLS ? v + row * v_stride + (size_t)h * V + min(first_col + small_e, V - 1)
                              : small_e == WIDE_COLS ? gate + row * gate_stride + h : beta + row * beta_stride + h;
@@ -260,6 +271,10 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
+    if (D < Dp) {
+        for (int i = threadIdx.x; i < 2 * WIDE_CH * row_floats; i += THREADS) stage[i] = 0.0f;
+        __syncthreads();
+    }
     const int chunks = (n + WIDE_CH - 1) / WIDE_CH;
     issue(0, 0);
     for (int c = 0; c < chunks; ++c) {
@@ -268,46 +283,105 @@ recurrence_wide_kernel(const float* __restrict__ q, const float* __restrict__ k,
         if (c + 1 < chunks) issue(c + 1, (c + 1) & 1);
         const float* buf = stage + (size_t)(c & 1) * WIDE_CH * row_floats;
         const int rows = min(WIDE_CH, n - c * WIDE_CH);
-        for (int t = 0; t < rows; ++t) {
-            const float* rowp = buf + (size_t)t * row_floats;
-            float kk[PER], qq[PER];
-            read_run<PER>(rowp, lane, D, qq);
-            read_run<PER>(rowp + Dp, lane, D, kk);
-            float u = rowp[NV * Dp + warp];
-            const float raw = u;
-            float a = dec;
-            if (VEC) {
-                float gg[PER];
-                read_run<PER>(rowp + 2 * Dp, lane, D, gg);
+        if constexpr (MODE != M_DELTA && MODE != M_DELTA_VEC) {
+            // A whole group of rows has no condition within it, so that the reads of its rows run ahead of their sums.
+            auto group = [&](int t0, auto whole) {
+                float acc[WIDE_SUMS * CPW];          // [row][column]
 #pragma unroll
-                for (int i = 0; i < PER; ++i) S[i] *= gg[i];     // past D: S stays zero whatever the pad holds... the guard reads zeros there
+                for (int i = 0; i < WIDE_SUMS; ++i) {
+#pragma unroll
+                    for (int w = 0; w < CPW; ++w) acc[i * CPW + w] = 0.0f;
+                    if (!whole.value && t0 + i >= rows) continue;
+                    const float* rowp = buf + (size_t)(t0 + i) * row_floats;
+                    float kk[PER], qq[PER], gg[PER];
+                    read_run<PER>(rowp, lane, qq);
+                    read_run<PER>(rowp + Dp, lane, kk);
+                    if (VEC) read_run<PER>(rowp + 2 * Dp, lane, gg);
+                    float u[CPW];
+#pragma unroll
+                    for (int w = 0; w < CPW; ++w) u[w] = rowp[NV * Dp + warp * CPW + w];
+                    const float a = MODE == M_SCALED ? rowp[NV * Dp + WIDE_COLS] : dec;
+                    if (MODE == M_SCALED) {
+                        const float bt = rowp[NV * Dp + WIDE_COLS + 1];
+#pragma unroll
+                        for (int w = 0; w < CPW; ++w) u[w] *= bt;
+                    }
+#pragma unroll
+                    for (int d = 0; d < PER; ++d)
+#pragma unroll
+                        for (int w = 0; w < CPW; ++w) {
+                            S[w][d] = fmaf(VEC ? gg[d] : a, S[w][d], kk[d] * u[w]);
+                            acc[i * CPW + w] = fmaf(S[w][d], qq[d], acc[i * CPW + w]);
+                        }
+                }
+                // At each step a lane gives half of the sums it holds to its partner and takes the partner's share of the other
+                // half; when one is left, the lanes that hold the same one add theirs up.
+                int held = WIDE_SUMS * CPW, index = 0;
+#pragma unroll
+                for (int o = 16; o >= 1; o >>= 1) {
+                    if (held == 1) {
+                        acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], o);
+                        continue;
+                    }
+                    held >>= 1;
+                    const bool high = lane & o;
+                    if (high) index += held;
+#pragma unroll
+                    for (int i = 0; i < WIDE_SUMS * CPW / 2; ++i) {
+                        if (i >= held) continue;
+                        const float keep = high ? acc[i + held] : acc[i], give = high ? acc[i] : acc[i + held];
+                        acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                    }
+                }
+                const int t = t0 + index / CPW, w = index % CPW;
+                if (lane % (32 / (WIDE_SUMS * CPW)) == 0 && t < rows && col + w < V) {
+                    float sum = acc[0];
+                    if (MODE == M_SCALED) sum = fmaf(sk, buf[(size_t)t * row_floats + NV * Dp + warp * CPW + w], sum);
+                    out[(size_t)(a0 + c * WIDE_CH + t) * ((size_t)heads * V) + (size_t)h * V + col + w] = sum;
+                }
+            };
+            for (int t0 = 0; t0 < rows; t0 += WIDE_SUMS) {
+                if (t0 + WIDE_SUMS <= rows) group(t0, std::true_type{});
+                else group(t0, std::false_type{});
             }
-            if (MODE == M_DELTA || MODE == M_SCALED) a = rowp[NV * Dp + WIDE_COLS];
-            if (MODE == M_DELTA || MODE == M_DELTA_VEC) {
+        } else {
+            for (int t = 0; t < rows; ++t) {
+                const float* rowp = buf + (size_t)t * row_floats;
+                float kk[PER], qq[PER];
+                read_run<PER>(rowp, lane, qq);
+                read_run<PER>(rowp + Dp, lane, kk);
+                float u = rowp[NV * Dp + warp];
+                const float a = VEC ? 1.0f : rowp[NV * Dp + WIDE_COLS];
+                if (VEC) {
+                    float gg[PER];
+                    read_run<PER>(rowp + 2 * Dp, lane, gg);
+#pragma unroll
+                    for (int i = 0; i < PER; ++i) S[0][i] *= gg[i];     // past D everything is zero and stays so
+                }
                 float dot = 0.0f;
 #pragma unroll
-                for (int i = 0; i < PER; ++i) dot = fmaf(S[i], kk[i], dot);
+                for (int i = 0; i < PER; ++i) dot = fmaf(S[0][i], kk[i], dot);
                 dot = warp_sum(dot);
                 u = rowp[NV * Dp + WIDE_COLS + 1] * (u - a * dot);
-            }
-            if (MODE == M_SCALED) u = rowp[NV * Dp + WIDE_COLS + 1] * u;
-            float acc = 0.0f;
+                float acc = 0.0f;
 #pragma unroll
-            for (int i = 0; i < PER; ++i) {
-                S[i] = fmaf(a, S[i], kk[i] * u);
-                acc = fmaf(S[i], qq[i], acc);
+                for (int i = 0; i < PER; ++i) {
+                    S[0][i] = fmaf(a, S[0][i], kk[i] * u);
+                    acc = fmaf(S[0][i], qq[i], acc);
+                }
+                acc = warp_sum(acc);
+                if (col < V && lane == 0) out[(size_t)(a0 + c * WIDE_CH + t) * ((size_t)heads * V) + (size_t)h * V + col] = acc;
             }
-            acc = warp_sum(acc);
-            if (MODE == M_SCALED) acc = fmaf(sk, raw, acc);
-            if (live && lane == 0) out[(size_t)(a0 + c * WIDE_CH + t) * ((size_t)heads * V) + (size_t)h * V + j] = acc;
         }
     }
-    if (live) {
-        float* sout = state + (size_t)slot_out[r] * slot_floats + ((size_t)h * V + j) * D;
+#pragma unroll
+    for (int w = 0; w < CPW; ++w) {
+        if (col + w >= V) continue;
+        float* sout = state + (size_t)slot_out[r] * slot_floats + ((size_t)h * V + col + w) * D;
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
             const int d = lane * PER + i;
-            if (d < D) sout[d] = S[i];
+            if (d < D) sout[d] = S[w][i];
         }
     }
 }
@@ -412,9 +486,12 @@ channel_decay_kernel(float* __restrict__ proj, int stride, int rows, int low_off
     const int c = blockIdx.x * DECAY_THREADS + threadIdx.x;
     const int r0 = blockIdx.y * DECAY_ROWS, n = min(DECAY_ROWS, rows - r0);
     const float b = bias && c < channels ? bias[c] : 0.0f;
-    float z[DECAY_ROWS];
+    float z[DECAY_ROWS], qv[DECAY_ROWS];
 #pragma unroll
-    for (int r = 0; r < DECAY_ROWS; ++r) z[r] = b;
+    for (int r = 0; r < DECAY_ROWS; ++r) {
+        z[r] = b;
+        qv[r] = c < channels && r < n ? proj[(size_t)(r0 + r) * stride + q_off + c] : 0.0f;      // on its way during the sums
+    }
     for (int k0 = 0; k0 < rank; k0 += DECAY_RANK) {
         const int kn = min(DECAY_RANK, rank - k0);
         __syncthreads();
@@ -424,6 +501,7 @@ channel_decay_kernel(float* __restrict__ proj, int stride, int rows, int low_off
         }
         __syncthreads();
         if (c < channels)
+#pragma unroll 8
             for (int k = 0; k < kn; ++k) {
                 const float w = w2t[(size_t)(k0 + k) * channels + c];
 #pragma unroll
@@ -436,7 +514,7 @@ channel_decay_kernel(float* __restrict__ proj, int stride, int rows, int low_off
         if (r >= n) break;
         const float log_sigmoid = fminf(z[r], 0.0f) - log1pf(expf(-fabsf(z[r])));
         decay[(size_t)(r0 + r) * channels + c] = expf(log_sigmoid * inv_tau);
-        if (q_factor != 1.0f) proj[(size_t)(r0 + r) * stride + q_off + c] *= q_factor;
+        proj[(size_t)(r0 + r) * stride + q_off + c] = qv[r] * q_factor;
     }
 }
 
@@ -464,7 +542,7 @@ int launch_recurrence(int D, bool wide, int requests, cudaStream_t stream, const
         if (smem > 200 * 1024) return LLMX_ERR_UNSUPPORTED;                                                               \
         if (smem > 48 * 1024)                                                                                             \
             cudaFuncSetAttribute(recurrence_wide_kernel<P, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        launch_kernel(recurrence_wide_kernel<P, MODE>, dim3(requests, (unsigned)by), dim3(WIDE_THREADS), smem, stream, q, \
+        launch_kernel(recurrence_wide_kernel<P, MODE>, dim3(requests, (unsigned)by), dim3(wide_threads(MODE)), smem, stream, q, \
                       k, v, q_stride, k_stride, v_stride, decay, gate, beta, gate_stride, beta_stride, skip, state,      \
                       slot_floats, row_start, row_count, history, slot_in, slot_out, out, heads, qk_heads, D, V);       \
         return launch_status();                                                                                           \
